@@ -5,8 +5,8 @@
  * a LIST of layers — each a token mixer and an optional feed-forward between grouped RMS norms — where the mixers differ from
  * layer to layer and keep different per-request state:
  *   XOTB200_LM_MIX_LATENT_ATTN  attention over a compressed (latent) key/value row per token + one rotated key part shared by
- *                               all heads; options: query through a normed latent, rotation layout, sliding window, output gate;
- *                               state = the paged latent cache;
+ *                               all heads; options: query through a normed latent, rotation layout, sliding window, output gate,
+ *                               softmax sink; state = the paged latent cache;
  *   XOTB200_LM_MIX_DELTA_RULE   generalised delta-rule recurrence with per-channel decay and removal rate;
  *                               state = one fp32 matrix per head, request and layer;
  *   XOTB200_LM_MIX_ATTENTION    grouped-query attention over a paged cache of (normed) keys and values; options: projection
@@ -24,8 +24,10 @@
  * mix_scale * first + par_scale * second.
  * A layer wraps its sublayers in grouped RMS norms before and after them, or reads the stream itself and closes with a layer norm
  * or an RMS norm, or — pre-norm with one-number weights — reads `streams` copies of the residual stream through hyper-connections
- * and passes every sublayer input through a short causal convolution that is added to it (xotb200_lm_cfg.block); its feed-forward is dense (relu^2 or xIELU) or a mixture of experts (gated silu or relu^2
- * experts, two routing rules, an optional shared expert: xotb200_lm_layer.ff_kind and the fields after it).
+ * and passes every sublayer input through a short causal convolution that is added to it, or — pre-norm with a Dynamic Tanh —
+ * norms every entry of the stream by itself (xotb200_lm_cfg.block); its feed-forward is dense (relu^2, xIELU, gelu, gated gelu) or a
+ * mixture of experts (gated silu, clamped gated or relu^2 experts, three routing rules, an optional shared expert:
+ * xotb200_lm_layer.ff_kind and the fields after it).  A layer may use another layer's weights (weights_of) with a cache / state of its own.
  * Every size and constant of a layer is a field of xotb200_lm_layer, so a model family is a table of layers, not code.
  *
  * Serving model: requests live in SLOTS (0 .. max_requests-1).  A step (xotb200_lm_step) takes a packed batch — for each
@@ -67,13 +69,19 @@ extern "C" {
 #define XOTB200_LM_FF_XIELU 1  /* W_down act(W_up h), act(z) = softplus(p) z^2 + z/2 (z > 0), (1/2 + softplus(q))(e^z - 1 - z) + z/2 (z <= 0);
                                   p, q = the two entries of l<i>.mlp.act                                                         */
 #define XOTB200_LM_FF_GELU 3   /* W_down gelu(W_up h), the exact gelu z (1 + erf(z / sqrt 2)) / 2                               */
+#define XOTB200_LM_FF_GELU_GATED 4 /* W_down (gelu_tanh(W_gate h) * W_up h), the tanh form of gelu                                */
 #define XOTB200_LM_FF_MOE 2    /* mixture of experts; expert form, routing rule and shared expert: expert_act, router_kind, shared_ff */
 
 #define XOTB200_LM_EXPERT_SILU_GATED 0 /* expert = W_down (silu(W_gate h) * W_up h)                                              */
 #define XOTB200_LM_EXPERT_RELU2 1      /* expert = W_down relu(W_up h)^2  (no gate matrix)                                       */
+#define XOTB200_LM_EXPERT_CLAMPED_GLU 2 /* expert = W_down (g sigmoid(slope g) (u + 1)), g = min(W_gate h, limit), u = W_up h clamped to
+                                           [-limit, limit]  (expert_limit, expert_slope)                                          */
 
 #define XOTB200_LM_ROUTER_SOFTMAX_ALL 0 /* scores = softmax over all experts; group-limited top-k; weights = the chosen scores     */
 #define XOTB200_LM_ROUTER_TOPK_SOFTMAX 1 /* the `top` largest logits (W_router h + router.b) are chosen; weights = softmax over them */
+#define XOTB200_LM_ROUTER_SIGMOID_GROUPS 2 /* scores s = sigmoid(W_router h), choice scores s + correction; groups scored by the sum of their
+                                              group_best largest choice scores; the `top` largest choice scores of the kept groups;
+                                              weights = router_scale * s / (sum of the chosen s)                                  */
 
 #define XOTB200_LM_BLOCK_GROUP_RMS 0  /* x += norm1b(mixer(norm1(x))): grouped RMS norms before and after every sublayer          */
 #define XOTB200_LM_BLOCK_POST_LN 1    /* x += LN(mixer(x)): the sublayer reads the stream itself, layer norm (weight + bias) on its output */
@@ -82,6 +90,9 @@ extern "C" {
 #define XOTB200_LM_BLOCK_PRE_SCALAR 3  /* x += mult * sublayer(c(rms(x) * g)): pre-norm whose weight is ONE number, c(h) = h + causal
                                          convolution of h over time (canon_taps; 0 = none); with streams > 0 the stream is kept in
                                          `streams` copies mixed by hyper-connections (below); embedding and final norm of the same kind */
+
+#define XOTB200_LM_BLOCK_PRE_DYT 4     /* x += ls * sublayer(tanh(alpha x) * w + b): pre-norm by a Dynamic Tanh (no statistic of the row), the
+                                         sublayer's result scaled entry by entry when layer_scale; the final norm of the same kind      */
 
 #define XOTB200_LM_QKNORM_NONE 0
 #define XOTB200_LM_QKNORM_HEAD 1      /* RMS norm of every query / key head, one weight of size dim shared by the heads                 */
@@ -179,6 +190,15 @@ typedef struct xotb200_lm_layer {
   float par_gate_cap;
   float mix_scale;      /* the layer's mixer output = mix_scale * this mixer (0 = 1) + par_scale * the second                    */
   float par_scale;
+  /* -- a layer that uses another layer's weights; further options of FF_MOE ------------------------------------------------------ */
+  int32_t weights_of;     /* -1 = own tensors; else the (global) index of the layer whose tensors it uses (every other field equal to that
+                             layer's, which has tensors of its own); cache and state are the layer's own.  `sink` is an option of
+                             MIX_LATENT_ATTN too. */
+  float expert_limit;     /* EXPERT_CLAMPED_GLU: bound of gate and up values ...                                    */
+  float expert_slope;     /* ... and slope of the gate's sigmoid                                                    */
+  int32_t router_correction; /* ROUTER_SIGMOID_GROUPS: 1 = choice scores have a correction per expert (mlp.correction)   */
+  int32_t group_best;     /* ROUTER_SIGMOID_GROUPS: how many of a group's largest choice scores make its score (1 or 2) */
+  float router_scale;     /* ROUTER_SIGMOID_GROUPS: factor of the normalised weights                                */
 } xotb200_lm_layer;
 
 typedef struct xotb200_lm_cfg {
@@ -205,6 +225,8 @@ typedef struct xotb200_lm_cfg {
   int32_t streams;
   int32_t canon_taps;    /* > 0: taps of the convolution on every sublayer input (l<i>.canon<q> [width, taps], last tap = current token) */
   float residual_mult;   /* 0 = 1                                                                                                   */
+  int32_t layer_scale;   /* BLOCK_PRE_DYT: 1 = a sublayer's result is multiplied entry by entry by l<i>.ls1 / ls2 before the sum          */
+  int32_t tied_head;     /* 1 = the logits use the embedding table (no tensor `head`)                                               */
 } xotb200_lm_cfg;
 
 typedef struct xotb200_lm xotb200_lm;
@@ -226,6 +248,8 @@ int xotb200_lm_destroy(xotb200_lm* e);
  * have no gate matrix.
  * BLOCK_PRE_SCALAR models: embed.norm, final.norm, l<i>.norm1 / norm2 (one number each), l<i>.canon1 / canon2, l<i>.hc1 / hc2 .in / .out /
  * .mix; MIX_ATTENTION with QKNORM_HEAD_PLAIN has no norm weights; MIX_MATRIX_LSTM <t> in {q, k, v, g, i, i.b, f, f.b, norm, o};
+ * BLOCK_PRE_DYT models: norm weights <norm>, <norm>.alpha (one number), <norm>.b for l<i>.norm1 / norm2 and final.norm; l<i>.ls1 / ls2;
+ * MIX_LATENT_ATTN with a sink: sink [heads]; FF_GELU_GATED: mlp.gate / up / down; ROUTER_SIGMOID_GROUPS: mlp.correction [experts].
  * MIX_MAMBA2 <t> in {in, conv, conv.b, dt_bias, A_log, D, norm, o}; a layer with two mixers names them l<i>.mix.left.<t> / .right.<t>.
  * xotb200_lm_load_dir reads every *.safetensors of the directory (BF16 tensors) and is STRICT: a tensor of this shard that is
  * missing, has another shape or dtype, or an unknown tensor of an owned layer, is an error. */

@@ -80,6 +80,8 @@ struct Dest {
 struct LmLayer {
   xotb200_lm_layer s;
   size_t norm1, norm1b, norm2, norm2b;                 // element offsets into the blob
+  size_t norm1a = 0, norm2a = 0, ls1 = 0, ls2 = 0;     // Dynamic-Tanh block: the norms' scalars, the layer scales
+  size_t state_begin = 0, state_size = 0;              // floats of a slot's state block that belong to this layer
   size_t w_in;                                         // concatenated input projections [n_in, D]
   int n_in;
   int c_q, c_kv, c_g;                                  // latent attention: columns of the projection output
@@ -99,7 +101,7 @@ struct LmLayer {
   int c_b = 0, conv_ch = 0;
   size_t conv_off = 0;                                 // float offset of the filter inputs inside a slot's state block
   // feed-forward forms: xIELU parameters; mixture of experts: router [E, D], experts' [E][2 F, D] (gate rows, up rows) and [E][D, F]
-  size_t act_p = 0, router = 0, router_b = 0, w_gu = 0, w_edown = 0;   // a shared expert's matrices are `up` / `down`
+  size_t act_p = 0, router = 0, router_b = 0, correction = 0, w_gu = 0, w_edown = 0;   // a shared expert's matrices are `up` / `down`
   // matrix LSTM: gate biases, float offset of the running maxima in a slot's block; state-space layer: filter bias, skip weights
   size_t i_b = 0, f_b = 0, conv_b = 0, d_skip = 0, m_off = 0, n_off = 0;
   int c_i = 0, c_f = 0, c_z = 0, c_dt = 0;
@@ -162,7 +164,10 @@ struct xotb200_lm {
                                                        // before its convolution, matrix-LSTM decay / input weight / floor / n . q per (row, head)
   int max_heads_rec = 0;
   bool pre_scalar = false;
-  size_t final_norm_b = 0, pos_table = 0;
+  bool pre_dyt = false;
+  size_t final_norm_b = 0, final_norm_a = 0, pos_table = 0;
+  const EpiArgs* close = nullptr;                      // set by a block form whose sublayers close themselves in their last kernel; NULL: they write y
+  bool closed = false;                                 // the sublayer that ran has done so
   void* oh2 = nullptr;                                 // the second mixer's operand of its output product
   void *h = nullptr, *cqn = nullptr, *qn = nullptr, *olat = nullptr, *oh = nullptr, *act = nullptr, *th = nullptr, *hw = nullptr;
   void *q16 = nullptr, *cbuf = nullptr, *knx = nullptr, *vxx = nullptr;   // expanded prompt attention (bf16)
@@ -215,10 +220,11 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
   auto take = [&](size_t n) { size_t o = cur; cur = align_up(cur + n, al); return o; };
   auto dest = [&](const std::string& name, size_t off, int rows, int cols, int row_off) { e->dests[name] = Dest{off, rows, cols, row_off, false}; };
   const bool post_ln = e->cfg.block == XOTB200_LM_BLOCK_POST_LN, post_rms = e->cfg.block == XOTB200_LM_BLOCK_POST_RMS;
-  const bool pre_scalar = e->cfg.block == XOTB200_LM_BLOCK_PRE_SCALAR;
+  const bool pre_scalar = e->cfg.block == XOTB200_LM_BLOCK_PRE_SCALAR, pre_dyt = e->cfg.block == XOTB200_LM_BLOCK_PRE_DYT;
   const int NW = pre_scalar ? 1 : D;                   // entries of a block norm's weight
   const int S = e->cfg.streams, CT = e->cfg.canon_taps;
   e->pre_scalar = pre_scalar;
+  e->pre_dyt = pre_dyt;
   // what a sublayer of the pre-scalar block owns besides its norm: input convolution and hyper-connection coefficients
   auto sublayer_extras = [&](LmLayer& L, const std::string& p, int q) {
     const std::string n = std::to_string(q + 1);
@@ -235,7 +241,13 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
   };
   // the weight after a sublayer: a second grouped RMS norm ("norm1b"), or the bias of the closing layer norm ("norm1.b"); a closing
   // RMS norm has one weight only
-  const std::string nb = post_ln ? ".b" : "b";
+  const std::string nb = post_ln || pre_dyt ? ".b" : "b";
+  // a Dynamic Tanh also has a scalar; the sublayer behind it a scale
+  auto dyt_extras = [&](const std::string& p, const std::string& n, size_t& alpha, size_t& ls) {
+    alpha = take(1); dest(p + "norm" + n + ".alpha", alpha, 1, 1, 0);
+    if (e->cfg.layer_scale) { ls = take(D); dest(p + "ls" + n, ls, 1, D, 0); }
+  };
+  std::map<int, size_t> owners;                        // layer that names the tensors -> local index of the first local layer that uses them
   if (e->first) {
     e->embed = take((size_t)V * D); dest("embed", e->embed, V, D, 0);
     if (e->cfg.embed_norm) { e->embed_norm = take(NW); dest("embed.norm", e->embed_norm, 1, NW, 0); }
@@ -245,11 +257,39 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
     LmLayer L{};
     L.s = all[li];
     const xotb200_lm_layer& s = L.s;
-    const std::string p = "l" + std::to_string(li) + ".";
+    const int own_li = s.weights_of >= 0 ? s.weights_of : li;
+    if (s.weights_of >= 0) {
+      REQUIRE(own_li < e->cfg.n_layers && all[own_li].weights_of < 0, "layer %d uses the weights of layer %d, which has no tensors of its own", li, own_li);
+      xotb200_lm_layer same = all[own_li];
+      same.weights_of = s.weights_of;
+      REQUIRE(memcmp(&same, &s, sizeof(same)) == 0, "layer %d uses the weights of layer %d but has other sizes or constants", li, own_li);
+    }
+    const auto known = owners.find(own_li);
+    if (known != owners.end()) {
+      // the tensors are laid out already: same offsets, state and cache of its own
+      LmLayer C = e->layers[known->second];
+      const size_t shift = e->state_floats - C.state_begin;
+      auto move_state = [&](LmLayer& X) {
+        X.state_off += shift; X.conv_off += shift; X.m_off += shift; X.n_off += shift;
+        X.canon_off[0] += shift; X.canon_off[1] += shift;
+      };
+      move_state(C);
+      for (LmLayer& X : C.par) move_state(X);
+      C.state_begin += shift;
+      e->state_floats += C.state_size;
+      C.s = s;
+      if (s.mixer == XOTB200_LM_MIX_ATTENTION && s.kv_from < 0) C.kv_src = li - e->cfg.start_layer;
+      e->layers.push_back(C);
+      continue;
+    }
+    owners[own_li] = e->layers.size();
+    L.state_begin = e->state_floats;
+    const std::string p = "l" + std::to_string(own_li) + ".";
     REQUIRE(s.heads >= 1 && s.dim >= 1, "layer %d: heads and dim must be positive", li);
     L.norm1 = take(NW); dest(p + "norm1", L.norm1, 1, NW, 0);
     if (!post_rms && !pre_scalar) { L.norm1b = take(D); dest(p + "norm1" + nb, L.norm1b, 1, D, 0); }
     if (pre_scalar) sublayer_extras(L, p, 0);
+    if (pre_dyt) dyt_extras(p, "1", L.norm1a, L.ls1);
     // one mixer: its projection columns start at column cb of the layer's projection output; `shared`: the projection matrix of
     // the layer's mixers is one allocation (w_shared) and this mixer's rows follow the first mixer's
     auto layout_mixer = [&](LmLayer& L, const std::string& mp, int cb, bool shared, size_t w_shared) -> int {
@@ -275,6 +315,7 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
       dest(mp + "dkv", L.w_in, R + dr, D, L.c_kv);
       if (s.out_gate) dest(mp + "g", L.w_in, H, D, L.c_g);
       L.dkv_norm = take(R); dest(mp + "dkv.norm", L.dkv_norm, 1, R, 0);
+      if (s.sink) { L.sink = take(H); dest(mp + "sink", L.sink, 1, H, 0); }
       // W_uk is kept per head as [R, dn]: the absorption product q~ = W_uk[h]^T q then reads it K-major like every other weight
       L.uk = take((size_t)H * dn * R); dest(mp + "uk", L.uk, H * dn, R, 0); e->dests[mp + "uk"].tr_heads = H;
       L.uk_rows = take((size_t)H * dn * R); e->dests[mp + "uk"].has2 = true; e->dests[mp + "uk"].elem_off2 = L.uk_rows;
@@ -496,6 +537,7 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
       L.norm2 = take(NW); dest(p + "norm2", L.norm2, 1, NW, 0);
       if (!post_rms && !pre_scalar) { L.norm2b = take(D); dest(p + "norm2" + nb, L.norm2b, 1, D, 0); }
       if (pre_scalar) sublayer_extras(L, p, 1);
+      if (pre_dyt) dyt_extras(p, "2", L.norm2a, L.ls2);
     }
     if (s.ff_kind == XOTB200_LM_FF_MOE && has_ff) {
       const int E = s.experts, F = s.expert_ff;
@@ -503,12 +545,16 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
       if (s.groups > 1)
         REQUIRE(E % s.groups == 0 && s.groups_keep >= 1 && s.groups_keep <= s.groups && s.groups_keep * (E / s.groups) >= s.top,
                 "layer %d: %d experts in %d groups of which %d are kept cannot give %d experts per token", li, E, s.groups, s.groups_keep, s.top);
-      REQUIRE(s.expert_act == XOTB200_LM_EXPERT_SILU_GATED || s.expert_act == XOTB200_LM_EXPERT_RELU2, "layer %d: unknown expert form %d", li, s.expert_act);
-      REQUIRE(s.router_kind == XOTB200_LM_ROUTER_SOFTMAX_ALL || s.router_kind == XOTB200_LM_ROUTER_TOPK_SOFTMAX, "layer %d: unknown routing rule %d", li, s.router_kind);
+      REQUIRE(s.expert_act >= XOTB200_LM_EXPERT_SILU_GATED && s.expert_act <= XOTB200_LM_EXPERT_CLAMPED_GLU, "layer %d: unknown expert form %d", li, s.expert_act);
+      REQUIRE(s.expert_act != XOTB200_LM_EXPERT_CLAMPED_GLU || s.expert_limit > 0.f, "layer %d: the clamped experts need a positive limit", li);
+      REQUIRE(s.router_kind >= XOTB200_LM_ROUTER_SOFTMAX_ALL && s.router_kind <= XOTB200_LM_ROUTER_SIGMOID_GROUPS, "layer %d: unknown routing rule %d", li, s.router_kind);
+      REQUIRE(s.router_kind != XOTB200_LM_ROUTER_SIGMOID_GROUPS || s.groups <= 1 || s.group_best == 1 || s.group_best == 2,
+              "layer %d: a group is scored by its best or its two best experts, not %d", li, s.group_best);
       REQUIRE(s.shared_ff >= 0, "layer %d: negative size of the shared expert", li);
-      const bool gated = s.expert_act == XOTB200_LM_EXPERT_SILU_GATED;
+      const bool gated = s.expert_act != XOTB200_LM_EXPERT_RELU2;
       L.router = take((size_t)E * D); dest(p + "mlp.router", L.router, E, D, 0);
       if (s.router_bias) { L.router_b = take(E); dest(p + "mlp.router.b", L.router_b, 1, E, 0); }
+      if (s.router_correction) { L.correction = take(E); dest(p + "mlp.correction", L.correction, 1, E, 0); }
       L.w_gu = take((size_t)E * (gated ? 2 : 1) * F * D);
       L.w_edown = take((size_t)E * D * F);
       for (int x = 0; x < E; ++x) {
@@ -532,19 +578,30 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
       e->max_eff = std::max(e->max_eff, F);
       e->max_experts = std::max(e->max_experts, E);
     } else if (has_ff) {
-      REQUIRE(s.ff_kind == XOTB200_LM_FF_RELU2 || s.ff_kind == XOTB200_LM_FF_XIELU || s.ff_kind == XOTB200_LM_FF_GELU, "layer %d: unknown feed-forward kind %d", li,
-              s.ff_kind);
-      L.up = take((size_t)s.ff * D); dest(p + "mlp.up", L.up, s.ff, D, 0);
+      REQUIRE(s.ff_kind == XOTB200_LM_FF_RELU2 || s.ff_kind == XOTB200_LM_FF_XIELU || s.ff_kind == XOTB200_LM_FF_GELU || s.ff_kind == XOTB200_LM_FF_GELU_GATED,
+              "layer %d: unknown feed-forward kind %d", li, s.ff_kind);
+      if (s.ff_kind == XOTB200_LM_FF_GELU_GATED) {             // gate and up rows as one matrix (see glu_gate_row)
+        L.up = take((size_t)2 * s.ff * D);
+        dest(p + "mlp.gate", L.up, s.ff, D, 0);
+        dest(p + "mlp.up", L.up, s.ff, D, s.ff % 8 ? s.ff : 0);
+        if (s.ff % 8 == 0) { e->dests[p + "mlp.gate"].il8 = 0; e->dests[p + "mlp.up"].il8 = 1; }
+      } else {
+        L.up = take((size_t)s.ff * D); dest(p + "mlp.up", L.up, s.ff, D, 0);
+      }
       L.down = take((size_t)D * s.ff); dest(p + "mlp.down", L.down, D, s.ff, 0);
       if (s.ff_kind == XOTB200_LM_FF_XIELU) { L.act_p = take(2); dest(p + "mlp.act", L.act_p, 1, 2, 0); }
       e->max_ff = std::max(e->max_ff, s.ff);
     }
+    L.state_size = e->state_floats - L.state_begin;
     e->layers.push_back(L);
   }
   if (e->last) {
     e->final_norm = take(NW); dest("final.norm", e->final_norm, 1, NW, 0);
-    if (post_ln) { e->final_norm_b = take(D); dest("final.norm.b", e->final_norm_b, 1, D, 0); }   // a final RMS norm has a weight only
-    e->head = take((size_t)V * D); dest("head", e->head, V, D, 0);
+    if (post_ln || pre_dyt) { e->final_norm_b = take(D); dest("final.norm.b", e->final_norm_b, 1, D, 0); }   // a final RMS norm has a weight only
+    if (pre_dyt) { e->final_norm_a = take(1); dest("final.norm.alpha", e->final_norm_a, 1, 1, 0); }
+    if (!e->cfg.tied_head) { e->head = take((size_t)V * D); dest("head", e->head, V, D, 0); }
+    else if (e->first) e->head = e->embed;
+    else { e->head = take((size_t)V * D); dest("embed", e->head, V, D, 0); }   // the last of several shards holds its own copy of the table
   }
   e->blob_elems = cur;
   return 0;
@@ -587,7 +644,7 @@ static int upload_tensor(xotb200_lm* e, Dest& d, const void* host_bf16) {
 // does a tensor name belong to this shard? (so that an unknown name there is an error, and anything else is skipped)
 static bool owned_name(const xotb200_lm* e, const std::string& name) {
   if (name == "embed" || name == "pos" || name == "embed.norm") return e->first;
-  if (name == "head" || name == "final.norm" || name == "final.norm.b") return e->last;
+  if (name == "head" || name == "final.norm" || name == "final.norm.b" || name == "final.norm.alpha") return e->last;
   if (name.size() > 1 && name[0] == 'l' && isdigit((unsigned char)name[1])) {
     const int li = atoi(name.c_str() + 1);
     return li >= e->cfg.start_layer && li <= e->cfg.end_layer;
@@ -651,11 +708,11 @@ static int launch_ltc(xotb200_lm* e, const CUtensorMap& ma, const CUtensorMap& m
 // 1 = launched, 0 = not eligible (the caller falls back), < 0 = error
 template <typename TC, int EPI>
 static int product_tc(xotb200_lm* e, const bf16* A, long lda, long a_batch, const bf16* B, long ldb, long b_batch, TC* C, long ldc, long c_batch, int M,
-                      int N, int K, int batch, const void* epi) {
+                      int N, int K, int batch, const EpiArgs& epi) {
   const int nt = (N > 64 && M > LTC_M) ? 128 : 64;   // one row tile: narrower column tiles, twice the CTAs streaming weights
   CUtensorMap ma, mb;
   if (!make_map3(&ma, A, M, K, lda, a_batch, batch, LTC_M) || !make_map3(&mb, B, N, K, ldb, b_batch, batch, nt)) return 0;
-  LtcArgs a{M, N, K, C, ldc, c_batch, e->d_err, static_cast<const bf16*>(epi), nullptr, 0};
+  LtcArgs a{M, N, K, C, ldc, c_batch, e->d_err, epi, nullptr, 0};
   if (nt == 128) TRY((launch_ltc<128, EPI, TC>(e, ma, mb, a, batch)));
   else TRY((launch_ltc<64, EPI, TC>(e, ma, mb, a, batch)));
   return 1;
@@ -663,12 +720,12 @@ static int product_tc(xotb200_lm* e, const bf16* A, long lda, long a_batch, cons
 
 template <typename TA, typename TB, typename TC, int EPI>
 static int product(xotb200_lm* e, const TA* A, long lda, long a_batch, const TB* B, long sbn, long sbk, long b_batch, TC* C, long ldc, long c_batch,
-                   int M, int N, int K, int batch, const void* epi = nullptr) {
+                   int M, int N, int K, int batch, const EpiArgs& epi = EpiArgs{}) {
   if (M == 0 || N == 0) return 0;
   const size_t smem = (size_t)M * K * 4;
-  if constexpr (std::is_same<TA, bf16>::value && std::is_same<TB, bf16>::value && (EPI == 0 || !std::is_same<TC, float>::value)) {
+  if constexpr (std::is_same<TA, bf16>::value && std::is_same<TB, bf16>::value && (EPI == EPI_NONE || EPI == EPI_CLOSE || !std::is_same<TC, float>::value)) {
     // 16-bit operands with more rows than the decode kernel takes: the tensor cores, when the operands can be described to TMA
-    if (sbk == 1 && ((e->gemm_mode == 0 && M > GEMV_MAX_ROWS) || e->gemm_mode == 2)) {
+    if (sbk == 1 && (!epi_is_glu(EPI) || epi.il8) && ((e->gemm_mode == 0 && M > GEMV_MAX_ROWS) || e->gemm_mode == 2)) {
       const int r = product_tc<TC, EPI>(e, A, lda, a_batch, B, sbn, b_batch, C, ldc, c_batch, M, N, K, batch, epi);
       if (r != 0) return r < 0 ? r : 0;
     }
@@ -684,7 +741,7 @@ static int product(xotb200_lm* e, const TA* A, long lda, long a_batch, const TB*
     auto kern = gemv_rows_kernel<TA, TB, TC, EPI, MR>;                                                                         \
     TRY(opt_in_smem(kern, sm));                                                                                                \
     kern<<<dim3(blocks, 1, batch), 256, sm, e->stream>>>(A, lda, a_batch, B, sbn, b_batch, C, ldc, c_batch, M, N, K, wsplit,    \
-                                                         static_cast<const TB*>(epi));                                        \
+                                                         epi);                                                                \
   } while (0)
     if (M == 1) LAUNCH_GEMV(1);
     else if (M == 2) LAUNCH_GEMV(2);
@@ -693,11 +750,24 @@ static int product(xotb200_lm* e, const TA* A, long lda, long a_batch, const TB*
 #undef LAUNCH_GEMV
   } else {
     gemm_tiled_kernel<TA, TB, TC, EPI><<<dim3(cdiv(N, 64), cdiv(M, 64), batch), 256, 0, e->stream>>>(A, lda, a_batch, B, sbn, sbk, b_batch, C, ldc,
-                                                                                                  c_batch, M, N, K, static_cast<const TB*>(epi));
+                                                                                                  c_batch, M, N, K, epi);
   }
   CK(cudaGetLastError());
   e->launches++;
   return 0;
+}
+
+// The last product of a sublayer, y [M, D] = A W^T with D the model's width: into yout, or — under a block form that closes its sublayers
+// itself — straight into the stream and the next operand.
+template <typename T>
+static int output_product(xotb200_lm* e, const T* A, size_t w, int K, float* yout, int M) {
+  const int D = e->cfg.width;
+  if (e->close) {
+    TRY((product<T, T, float, EPI_CLOSE>(e, A, K, 0, at<T>(e, w), K, 1, 0, yout, D, 0, M, D, K, 1, *e->close)));
+    e->closed = true;
+    return 0;
+  }
+  return product<T, T, float, EPI_NONE>(e, A, K, 0, at<T>(e, w), K, 1, 0, yout, D, 0, M, D, K, 1);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
@@ -819,6 +889,23 @@ struct StepPlan {
   bool any_short = true;                               // some request goes through the absorbed kernel
 };
 
+// rows of one request that share a CTA of the absorbed attention kernel: about 32 (row, head) pairs
+static int latent_rows_per_item(const xotb200_lm_layer& s) { return std::max(1, 32 / s.heads); }
+// warps of its CTA (one per pair): the widest accumulator variant needs 70 registers, 16 warps at most
+static int latent_item_warps(const xotb200_lm_layer& s, int pairs) { return std::min(s.kv_rank > 256 ? 16 : 32, pairs); }
+
+// Few work items (decoding): the keys are cut into runs so that the GPU is filled; each run at least one 32-key tile.
+// Returns the number of runs and their length.
+static int latent_key_runs(const xotb200_lm* e, const xotb200_lm_layer& s, int n_items, int max_len, int* run) {
+  const int qpi = latent_rows_per_item(s), pairs = qpi * s.heads, ytiles = cdiv(pairs, latent_item_warps(s, pairs));
+  const int span = std::max(1, s.window > 0 ? std::min(max_len, s.window + qpi) : max_len);
+  int splits = 1;
+  const long ctas = (long)n_items * ytiles;
+  if (ctas > 0 && ctas < e->sm_count) splits = std::max(1, std::min(std::min(32, cdiv(span, 32)), cdiv(2 * e->sm_count, ctas)));
+  *run = cdiv(cdiv(span, splits), 32) * 32;
+  return cdiv(span, *run);
+}
+
 template <typename T>
 static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
   const xotb200_lm_layer& s = L.s;
@@ -838,49 +925,41 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
     q_ld = HQ;
   }
   const Paging pg{e->d_table, e->pages_per_slot, e->page_size};
-  latent_append_kernel<T><<<cdiv(M, 8), 256, 0, e->stream>>>(e->proj, L.n_in, L.c_kv, R, dr, at<T>(e, L.dkv_norm), eps, L.freqs, s.rot_dims, s.rot_layout,
-                                                             sp.row_slot, sp.row_pos, pg, static_cast<T*>(L.pool), M);
-  CK(cudaGetLastError());
-  e->launches++;
   // ---- which rows take which form
   const StepPlan::Flash* fl = nullptr;
   if constexpr (std::is_same<T, bf16>::value) {
     auto f = sp.flash.find(s.window);
     if (f != sp.flash.end() && f->second.n_tiles > 0) fl = &f->second;
   }
+  const bool absorbed = sp.any_short || !fl;
+  latent_prepare_kernel<T><<<cdiv((long)M * (H + 1), 8), 256, 0, e->stream>>>(qraw, q_ld, H, dn, dr, e->proj, L.n_in, L.c_kv, R, at<T>(e, L.dkv_norm), eps, L.freqs,
+                                                                              s.rot_dims, s.rot_layout, sp.row_slot, sp.row_pos, pg, static_cast<T*>(L.pool),
+                                                                              absorbed ? static_cast<T*>(e->qn) : nullptr, e->qfull,
+                                                                              fl ? static_cast<bf16*>(e->q16) : nullptr, M);
+  CK(cudaGetLastError());
+  e->launches++;
   const float* gate = s.out_gate ? e->proj : nullptr;
-  if (sp.any_short || !fl) {
+  const T* sink = s.sink ? at<T>(e, L.sink) : nullptr;
+  if (absorbed) {
     // absorbed form (few rows per request, and everything in the 32-bit mode)
-    query_split_kernel<T><<<cdiv((long)M * H, 8), 256, 0, e->stream>>>(qraw, q_ld, 0, H, dn, dr, R, L.freqs, s.rot_dims, s.rot_layout, sp.row_pos,
-                                                                        static_cast<T*>(e->qn), e->qfull, M);
-    CK(cudaGetLastError());
-    e->launches++;
     // key absorption: qfull[m, h, 0:R] = sum_d qn[m, h, d] * W_uk[h][:, d]
     TRY((product<T, T, float, 0>(e, static_cast<T*>(e->qn), (long)H * dn, dn, at<T>(e, L.uk), dn, 1, (long)dn * R, e->qfull, (long)H * (R + dr), R + dr, M, R,
                                  dn, H)));
-    const int qpi = std::max(1, 32 / H);
+    const int qpi = latent_rows_per_item(s);
     const auto& it = sp.items.at(qpi);
     if (it.second > 0) {
-      const int pairs = qpi * H, nw = std::min(R > 256 ? 16 : 32, pairs);   // the widest accumulator variant needs 70 registers: 16 warps at most
+      const int pairs = qpi * H, nw = latent_item_warps(s, pairs);
       const size_t smem = ((size_t)32 * ((R + dr) | 1) + (size_t)nw * (R + dr)) * 4;
-      // few work items (decoding): cut the keys into runs so that the GPU is filled; each run at least one 32-key tile
-      const int span = s.window > 0 ? std::min(sp.max_len, s.window + qpi) : sp.max_len;
-      int splits = 1;
-      if (it.second * cdiv(pairs, nw) < e->sm_count)
-        splits = std::max(1, std::min(std::min(32, cdiv(span, 32)), cdiv(2 * e->sm_count, it.second * cdiv(pairs, nw))));
-      const int chunk = cdiv(cdiv(span, splits), 32) * 32;
-      splits = cdiv(span, chunk);
-      if (splits > 1) {
-        const size_t need = (size_t)M * H * splits * (2 + R);
-        if (need > e->part_cap) { drop_graphs(e); TRY(regrow(e->part, need * 4)); e->part_cap = need; }
-      }
+      int chunk = 0;
+      const int splits = latent_key_runs(e, s, it.second, sp.max_len, &chunk);
+      REQUIRE(splits == 1 || (size_t)M * H * splits * (2 + R) <= e->part_cap, "internal: the key-run buffer was not sized for this step");
       const dim3 grid(it.second, cdiv(pairs, nw), splits);
 #define LAUNCH_ATTN(NACC)                                                                                                                       \
   do {                                                                                                                                          \
     auto kern = latent_attention_kernel<T, NACC>;                                                                                               \
     TRY(opt_in_smem(kern, smem));                                                                                                               \
     kern<<<grid, nw * 32, smem, e->stream>>>(e->qfull, static_cast<const T*>(L.pool), pg, it.first, H, R, dr, s.scale, s.window, gate, L.n_in, \
-                                             L.c_g, static_cast<T*>(e->olat), chunk, e->part);                                                  \
+                                             L.c_g, sink, static_cast<T*>(e->olat), chunk, e->part);                                            \
   } while (0)
       if (R <= 64) LAUNCH_ATTN(2);
       else if (R <= 128) LAUNCH_ATTN(4);
@@ -890,7 +969,7 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
       CK(cudaGetLastError());
       e->launches++;
       if (splits > 1) {
-        latent_attention_combine_kernel<T><<<dim3(it.second, cdiv(pairs, 8)), 256, 0, e->stream>>>(e->part, it.first, H, R, splits, gate, L.n_in, L.c_g, static_cast<T*>(e->olat));
+        latent_attention_combine_kernel<T><<<dim3(it.second, cdiv(pairs, 8)), 256, 0, e->stream>>>(e->part, it.first, H, R, splits, gate, L.n_in, L.c_g, sink, static_cast<T*>(e->olat));
         CK(cudaGetLastError());
         e->launches++;
       }
@@ -903,11 +982,9 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
     if (fl) {
       // expanded form for the requests that bring many rows (it overwrites their rows of `oh`)
       bf16 *q16 = static_cast<bf16*>(e->q16), *cbuf = static_cast<bf16*>(e->cbuf), *knx = static_cast<bf16*>(e->knx), *vxx = static_cast<bf16*>(e->vxx);
-      query_rotate16_kernel<<<cdiv((long)M * H, 8), 256, 0, e->stream>>>(qraw, q_ld, H, dn, dr, L.freqs, s.rot_dims, s.rot_layout, sp.row_pos, q16, M);
-      CK(cudaGetLastError());
       latent_gather_kernel<bf16><<<dim3(cdiv(fl->max_keys, 8), fl->n_reqs), 256, 0, e->stream>>>(static_cast<const bf16*>(L.pool), pg, fl->reqs, R + dr, cbuf);
       CK(cudaGetLastError());
-      e->launches += 2;
+      e->launches++;
       TRY((product<bf16, bf16, bf16, 0>(e, cbuf, R + dr, 0, at<bf16>(e, L.uk_rows), R, 1, 0, knx, (long)H * dn, 0, fl->n_keys, H * dn, R, 1)));
       TRY((product<bf16, bf16, bf16, 0>(e, cbuf, R + dr, 0, at<bf16>(e, L.uv), R, 1, 0, vxx, (long)H * dv, 0, fl->n_keys, H * dv, R, 1)));
       const int dqp = (dn + dr + 15) & ~15, dvt = dv <= 64 ? 8 : 16;
@@ -917,7 +994,7 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
   do {                                                                                                                                            \
     auto kern = KERN;                                                                                                                             \
     TRY(opt_in_smem(kern, SMEM));                                                                                                                 \
-    kern<<<grid, 128, SMEM, e->stream>>>(q16, knx, cbuf, vxx, fl->tiles, H, dn, dr, dv, R, s.scale, s.window, gate, L.n_in, L.c_g,               \
+    kern<<<grid, 128, SMEM, e->stream>>>(q16, knx, cbuf, vxx, fl->tiles, H, dn, dr, dv, R, s.scale, s.window, gate, L.n_in, L.c_g, sink,         \
                                          static_cast<bf16*>(e->oh));                                                                              \
   } while (0)
       if (aligned) {   // whole 16-byte chunks: cp.async double buffering, ldmatrix fragments
@@ -936,7 +1013,7 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
     }
   }
   // the output projection
-  TRY((product<T, T, float, 0>(e, static_cast<T*>(e->oh), (long)H * dv, 0, at<T>(e, L.wo), (long)H * dv, 1, 0, e->y, D, 0, M, D, H * dv, 1)));
+  TRY(output_product<T>(e, static_cast<T*>(e->oh), L.wo, H * dv, e->y, M));
   return 0;
 }
 
@@ -994,7 +1071,7 @@ static int delta_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
                                                                                static_cast<T*>(e->oh), s.heads, s.vdim, e->cfg.norm_eps, M);
   CK(cudaGetLastError());
   e->launches++;
-  TRY((product<T, T, float, 0>(e, static_cast<T*>(e->oh), HD, 0, at<T>(e, L.wo), HD, 1, 0, e->y, D, 0, M, D, HD, 1)));
+  TRY(output_product<T>(e, static_cast<T*>(e->oh), L.wo, HD, e->y, M));
   return 0;
 }
 
@@ -1023,7 +1100,7 @@ static int gqa_key_runs(const xotb200_lm* e, const xotb200_lm_layer& s, int n_it
 template <typename T>
 static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout) {
   const xotb200_lm_layer& s = L.s;
-  const int D = e->cfg.width, M = sp.M, H = s.heads, G = s.kv_heads, dk = s.dim, dv = s.vdim, rep = H / G;
+  const int M = sp.M, H = s.heads, G = s.kv_heads, dk = s.dim, dv = s.vdim, rep = H / G;
   const bool own = s.kv_from < 0;
   const Paging pg{e->d_table, e->pages_per_slot, e->page_size};
   T* pool = static_cast<T*>(e->layers[L.kv_src].pool);
@@ -1119,7 +1196,7 @@ static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout)
       e->flash_launches++;
     }
   }
-  TRY((product<T, T, float, 0>(e, static_cast<T*>(e->oh), (long)H * dv, 0, at<T>(e, L.wo), (long)H * dv, 1, 0, yout, D, 0, M, D, H * dv, 1)));
+  TRY(output_product<T>(e, static_cast<T*>(e->oh), L.wo, H * dv, yout, M));
   return 0;
 }
 
@@ -1140,7 +1217,7 @@ static int filter_channels(xotb200_lm* e, LmLayer& L, const StepPlan& sp, int co
 template <typename T>
 static int gated_delta_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout, void* ohbuf) {
   const xotb200_lm_layer& s = L.s;
-  const int D = e->cfg.width, M = sp.M, H = s.heads, G = s.kv_heads, dk = s.dim, dv = s.vdim, C = L.conv_ch;
+  const int M = sp.M, H = s.heads, G = s.kv_heads, dk = s.dim, dv = s.vdim, C = L.conv_ch;
   TRY(filter_channels<T>(e, L, sp, L.c_r, C, nullptr));
   gated_delta_prepare_kernel<T><<<cdiv((long)M * H, 8), 256, 0, e->stream>>>(e->cvb, C, e->proj, L.ld_in, L.c_b, L.c_a, at<T>(e, L.a_log), at<T>(e, L.dt_bias), e->wlog,
                                                                             e->du, e->dau, e->dkk, e->drr, H, G, dk, M);
@@ -1151,7 +1228,7 @@ static int gated_delta_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, floa
                                                                        H, dv, e->cfg.norm_eps, M);
   CK(cudaGetLastError());
   e->launches++;
-  TRY((product<T, T, float, 0>(e, static_cast<T*>(ohbuf), (long)H * dv, 0, at<T>(e, L.wo), (long)H * dv, 1, 0, yout, D, 0, M, D, H * dv, 1)));
+  TRY(output_product<T>(e, static_cast<T*>(ohbuf), L.wo, H * dv, yout, M));
   return 0;
 }
 
@@ -1160,7 +1237,7 @@ static int gated_delta_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, floa
 template <typename T>
 static int matrix_lstm_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout, void* ohbuf) {
   const xotb200_lm_layer& s = L.s;
-  const int D = e->cfg.width, M = sp.M, H = s.heads, dk = s.dim, dv = s.vdim;
+  const int M = sp.M, H = s.heads, dk = s.dim, dv = s.vdim;
   mlstm_gates_kernel<T><<<cdiv((long)sp.n_seq * H, 4), 128, 0, e->stream>>>(e->proj, L.ld_in, L.c_i, L.c_f, at<T>(e, L.i_b), at<T>(e, L.f_b), s.gate_cap, sp.seqs, sp.n_seq, H,
                                                                           e->state + L.m_off, e->state_floats, e->gdec, e->ginw, e->gfloor);
   CK(cudaGetLastError());
@@ -1175,7 +1252,7 @@ static int matrix_lstm_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, floa
                                                                        static_cast<T*>(ohbuf), H, dv, e->cfg.norm_eps, M);
   CK(cudaGetLastError());
   e->launches++;
-  TRY((product<T, T, float, 0>(e, static_cast<T*>(ohbuf), (long)H * dv, 0, at<T>(e, L.wo), (long)H * dv, 1, 0, yout, D, 0, M, D, H * dv, 1)));
+  TRY(output_product<T>(e, static_cast<T*>(ohbuf), L.wo, H * dv, yout, M));
   return 0;
 }
 
@@ -1184,7 +1261,7 @@ static int matrix_lstm_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, floa
 template <typename T>
 static int mamba2_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout, void* ohbuf) {
   const xotb200_lm_layer& s = L.s;
-  const int D = e->cfg.width, M = sp.M, H = s.heads, G = s.kv_heads, N = s.dim, dv = s.vdim, C = L.conv_ch, inner = H * dv;
+  const int M = sp.M, H = s.heads, G = s.kv_heads, N = s.dim, dv = s.vdim, C = L.conv_ch, inner = H * dv;
   TRY(filter_channels<T>(e, L, sp, L.c_v, C, at<T>(e, L.conv_b)));
   mamba2_prepare_kernel<T><<<cdiv((long)M * H, 8), 256, 0, e->stream>>>(e->cvb, C, e->proj, L.ld_in, L.c_dt, at<T>(e, L.a_log), at<T>(e, L.dt_bias), e->wlog, e->dkk, e->drr,
                                                                        H, G, N, dv, M);
@@ -1200,7 +1277,7 @@ static int mamba2_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yo
   }
   CK(cudaGetLastError());
   e->launches++;
-  TRY((product<T, T, float, 0>(e, static_cast<T*>(ohbuf), (long)inner, 0, at<T>(e, L.wo), (long)inner, 1, 0, yout, D, 0, M, D, inner, 1)));
+  TRY(output_product<T>(e, static_cast<T*>(ohbuf), L.wo, inner, yout, M));
   return 0;
 }
 
@@ -1208,11 +1285,11 @@ static int mamba2_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yo
 // 1 = launched, 0 = the operands cannot be described to TMA
 template <int EPI, typename TC>
 static int grouped_product(xotb200_lm* e, const bf16* A, long lda, const bf16* B, long ldb, long b_batch, int n_batch, TC* C, long ldc, int m_pad, int N,
-                           int K, const int* tile_batch) {
+                           int K, const int* tile_batch, const EpiArgs& epi = EpiArgs{}) {
   const int nt = N > 64 ? 128 : 64;
   CUtensorMap ma, mb;
   if (!make_map3(&ma, A, m_pad, K, lda, 0, 1, LTC_M) || !make_map3(&mb, B, N, K, ldb, b_batch, n_batch, nt)) return 0;
-  LtcArgs a{m_pad, N, K, C, ldc, 0, e->d_err, nullptr, tile_batch, 1};
+  LtcArgs a{m_pad, N, K, C, ldc, 0, e->d_err, epi, tile_batch, 1};
   if (nt == 128) TRY((launch_ltc<128, EPI, TC>(e, ma, mb, a, 1)));
   else TRY((launch_ltc<64, EPI, TC>(e, ma, mb, a, 1)));
   return 1;
@@ -1232,7 +1309,12 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
   T* h = static_cast<T*>(e->h);
   if (s.ff_kind == XOTB200_LM_FF_MOE) {
     const int E = s.experts, F = s.expert_ff, top = s.top;
-    const bool gated = s.expert_act == XOTB200_LM_EXPERT_SILU_GATED;
+    const bool gated = s.expert_act != XOTB200_LM_EXPERT_RELU2;
+    EpiArgs glu;
+    glu.il8 = gated && F % 8 == 0 ? 1 : 0;
+    glu.limit = s.expert_limit;
+    glu.slope = s.expert_slope;
+    const EpiArgs close = e->close ? *e->close : EpiArgs{};
     const int Fs = s.shared_ff;
     const bool grouped_ok = std::is_same<T, bf16>::value && M >= MOE_GROUPED_MIN_ROWS && e->gemm_mode != 1 && F % 8 == 0 && D % 8 == 0;
     // Few rows (and the 32-bit mode): the shared expert rides along in the experts' row kernels — no launches and no pass over y of
@@ -1246,14 +1328,14 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
     }
     {
       auto kern = moe_router_kernel<T>;
-      const size_t rsm = ((size_t)((D + 3) & ~3) + E) * 4;
+      const size_t rsm = ((size_t)((D + 3) & ~3) + (s.router_kind == XOTB200_LM_ROUTER_SIGMOID_GROUPS ? 2 * E + std::max(1, s.groups) : E)) * 4;
       TRY(opt_in_smem(kern, rsm));
       kern<<<M, std::min(1024, std::max(64, cdiv(E, 2) * 32)), rsm, e->stream>>>(h, D, at<T>(e, L.router), s.router_bias ? at<T>(e, L.router_b) : nullptr,
-                                                                                 s.router_kind, E, s.groups, s.groups_keep, top, e->moe_ids, e->moe_wts, M);
+                                                                                 s.router_kind, E, s.groups, s.groups_keep, top, s.router_correction ? at<T>(e, L.correction) : nullptr,
+                                                                                 s.group_best, s.router_scale, e->moe_ids, e->moe_wts, M);
     }
     CK(cudaGetLastError());
     e->launches++;
-    const int il8 = gated && F % 8 == 0 ? 1 : 0;
     if constexpr (std::is_same<T, bf16>::value) {
       if (grouped_ok) {
         const int pairs = M * top, tiles = cdiv(pairs, LTC_M) + E, m_pad = tiles * LTC_M;
@@ -1266,15 +1348,19 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
         moe_scatter_kernel<bf16><<<cdiv(pairs, 8), 256, 0, e->stream>>>(h, D, e->moe_ids, pairs, top, starts, cursor, place, xg);
         CK(cudaGetLastError());
         e->launches += 3;
-        int r = gated ? grouped_product<3, bf16>(e, xg, D, at<bf16>(e, L.w_gu), D, (long)2 * F * D, E, static_cast<bf16*>(e->mact), F, m_pad, 2 * F, D, tile_expert)
-                      : grouped_product<1, bf16>(e, xg, D, at<bf16>(e, L.w_gu), D, (long)F * D, E, static_cast<bf16*>(e->mact), F, m_pad, F, D, tile_expert);
+        bf16* ma = static_cast<bf16*>(e->mact);
+        int r = s.expert_act == XOTB200_LM_EXPERT_CLAMPED_GLU
+                    ? grouped_product<EPI_CLAMPED_GLU, bf16>(e, xg, D, at<bf16>(e, L.w_gu), D, (long)2 * F * D, E, ma, F, m_pad, 2 * F, D, tile_expert, glu)
+                : gated ? grouped_product<EPI_SILU_GLU, bf16>(e, xg, D, at<bf16>(e, L.w_gu), D, (long)2 * F * D, E, ma, F, m_pad, 2 * F, D, tile_expert, glu)
+                        : grouped_product<EPI_RELU2, bf16>(e, xg, D, at<bf16>(e, L.w_gu), D, (long)F * D, E, ma, F, m_pad, F, D, tile_expert);
         if (r < 0) return r;
-        if (r == 1) r = grouped_product<0, float>(e, static_cast<bf16*>(e->mact), F, at<bf16>(e, L.w_edown), F, (long)D * F, E, e->moe_yg, D, m_pad, D, F, tile_expert);
+        if (r == 1) r = grouped_product<EPI_NONE, float>(e, ma, F, at<bf16>(e, L.w_edown), F, (long)D * F, E, e->moe_yg, D, m_pad, D, F, tile_expert);
         if (r < 0) return r;
         if (r == 1) {
-          moe_combine_kernel<<<M, 256, 0, e->stream>>>(e->moe_yg, place, e->moe_wts, top, D, shared, e->y);
+          moe_combine_kernel<bf16><<<M, 256, 0, e->stream>>>(e->moe_yg, place, e->moe_wts, top, D, shared, e->y, close);
           CK(cudaGetLastError());
           e->launches++;
+          e->closed = e->close != nullptr;
           return 0;
         }
       }
@@ -1284,7 +1370,7 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
       TRY(opt_in_smem(kern, (size_t)D * 4));
       // a warp takes two weight rows per pass with gated experts (a gate row and its up row), four with ungated ones
       kern<<<dim3(M, top + (ride ? 1 : 0), std::max(1, std::min(cdiv(std::max(F, ride ? Fs : 0), gated ? 8 : 32), M <= 16 ? 1024 : 16))), 256, (size_t)D * 4, e->stream>>>(
-          h, D, at<T>(e, L.w_gu), F, il8, gated ? 1 : 0, e->moe_ids, top, static_cast<T*>(e->mact), ride ? at<T>(e, L.up) : nullptr, Fs, static_cast<T*>(e->act));
+          h, D, at<T>(e, L.w_gu), F, s.expert_act == XOTB200_LM_EXPERT_CLAMPED_GLU ? 2 : gated ? 1 : 0, glu, e->moe_ids, top, static_cast<T*>(e->mact), ride ? at<T>(e, L.up) : nullptr, Fs, static_cast<T*>(e->act));
       CK(cudaGetLastError());
       e->launches++;
     }
@@ -1293,20 +1379,27 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
       const size_t dsm = ((size_t)top * F + (ride ? Fs + 4 : 0)) * 4;
       TRY(opt_in_smem(kern, dsm));
       kern<<<dim3(M, std::max(1, std::min(cdiv(D, 16), M <= 16 ? 1024 : 16))), 256, dsm, e->stream>>>(static_cast<T*>(e->mact), F, at<T>(e, L.w_edown), D, e->moe_ids, e->moe_wts, top,
-                                                                                                   shared, e->y, static_cast<T*>(e->act), ride ? at<T>(e, L.down) : nullptr, Fs);
+                                                                                                   shared, e->y, static_cast<T*>(e->act), ride ? at<T>(e, L.down) : nullptr, Fs, close);
       CK(cudaGetLastError());
       e->launches++;
+      e->closed = e->close != nullptr;
     }
     return 0;
   }
-  if (s.ff_kind == XOTB200_LM_FF_GELU)
-    TRY((product<T, T, T, 4>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, static_cast<T*>(e->act), s.ff, 0, M, s.ff, D, 1)));
-  else if (s.ff_kind == XOTB200_LM_FF_XIELU)
-    TRY((product<T, T, T, 2>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, static_cast<T*>(e->act), s.ff, 0, M, s.ff, D, 1, at<T>(e, L.act_p))));
-  else
-    TRY((product<T, T, T, 1>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, static_cast<T*>(e->act), s.ff, 0, M, s.ff, D, 1)));
-  TRY((product<T, T, float, 0>(e, static_cast<T*>(e->act), s.ff, 0, at<T>(e, L.down), s.ff, 1, 0, e->y, D, 0, M, D, s.ff, 1)));
-  return 0;
+  T* act = static_cast<T*>(e->act);
+  EpiArgs epi;
+  if (s.ff_kind == XOTB200_LM_FF_GELU_GATED) {
+    epi.il8 = s.ff % 8 == 0 ? 1 : 0;
+    TRY((product<T, T, T, EPI_GELU_GLU>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, act, s.ff, 0, M, 2 * s.ff, D, 1, epi)));
+  } else if (s.ff_kind == XOTB200_LM_FF_GELU) {
+    TRY((product<T, T, T, EPI_GELU>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, act, s.ff, 0, M, s.ff, D, 1)));
+  } else if (s.ff_kind == XOTB200_LM_FF_XIELU) {
+    epi.p = at<T>(e, L.act_p);
+    TRY((product<T, T, T, EPI_XIELU>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, act, s.ff, 0, M, s.ff, D, 1, epi)));
+  } else {
+    TRY((product<T, T, T, EPI_RELU2>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, act, s.ff, 0, M, s.ff, D, 1)));
+  }
+  return output_product<T>(e, act, L.down, s.ff, e->y, M);
 }
 
 template <typename T>
@@ -1482,6 +1575,66 @@ static int run_layers_pre_scalar(xotb200_lm* e, const StepPlan& sp, int n_want) 
   return 0;
 }
 
+// Pre-norm layers with a Dynamic Tanh: x += ls * sublayer(tanh(alpha x) * w + b).  Every entry of the stream is normed by itself, so the
+// last kernel of a sublayer — a product's epilogue, the experts' down or combine kernel — adds its result to the stream AND writes the
+// next sublayer's operand: between two sublayers nothing is launched.  A sublayer whose last kernel cannot do that is closed by
+// close_rows_kernel.
+template <typename T>
+static int run_layers_pre_dyt(xotb200_lm* e, const StepPlan& sp, int n_want) {
+  const int D = e->cfg.width, M = sp.M;
+  T* h = static_cast<T*>(e->h);
+  const int nt = std::min(256, std::max(32, cdiv(D, 32) * 32));
+  LmLayer& L0 = e->layers.front();
+  if (e->first) embed_dyt_rows_kernel<T><<<M, nt, 0, e->stream>>>(at<T>(e, e->embed), sp.tokens, at<T>(e, L0.norm1a), at<T>(e, L0.norm1), at<T>(e, L0.norm1b), e->x, h, D);
+  else dyt_rows_kernel<T><<<M, nt, 0, e->stream>>>(e->x, nullptr, at<T>(e, L0.norm1a), at<T>(e, L0.norm1), at<T>(e, L0.norm1b), h, D);
+  CK(cudaGetLastError());
+  e->launches++;
+  // runs one sublayer: `ls` scales its result; the norm that follows it (a = NULL: none) makes the next operand
+  EpiArgs close;
+  auto sublayer = [&](auto&& body, size_t ls, const LmLayer* next, int q) -> int {
+    close = EpiArgs{};
+    close.x = e->x;
+    close.ld = D;
+    if (e->cfg.layer_scale) close.ls = at<T>(e, ls);
+    if (next) {
+      close.h = h;
+      close.alpha = at<T>(e, q ? next->norm2a : next->norm1a);
+      close.w = at<T>(e, q ? next->norm2 : next->norm1);
+      close.b = at<T>(e, q ? next->norm2b : next->norm1b);
+    }
+    e->close = &close;
+    e->closed = false;
+    const int rc = body();
+    e->close = nullptr;
+    if (rc < 0) return rc;
+    if (!e->closed) {
+      close_rows_kernel<T><<<M, nt, 0, e->stream>>>(close, e->y, D);
+      CK(cudaGetLastError());
+      e->launches++;
+    }
+    return 0;
+  };
+  for (size_t li = 0; li < e->layers.size(); ++li) {
+    LmLayer& L = e->layers[li];
+    const LmLayer* after = li + 1 < e->layers.size() ? &e->layers[li + 1] : nullptr;
+    const bool ff = layer_has_ff(L.s);
+    TRY(sublayer([&]() { return run_mixer<T>(e, L, sp); }, L.ls1, ff ? &L : after, ff ? 1 : 0));
+    if (ff) TRY(sublayer([&]() { return feed_forward<T>(e, L, sp); }, L.ls2, after, 0));
+    if (e->trace) CK(cudaMemcpyAsync(e->trace_buf + li * (size_t)M * D, e->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, e->stream));
+  }
+  if (e->trace) e->trace_floats = e->layers.size() * (size_t)M * D;
+  if (e->last && n_want > 0) {
+    T* hw = static_cast<T*>(e->hw);
+    dyt_rows_kernel<T><<<n_want, nt, 0, e->stream>>>(e->x, sp.want, at<T>(e, e->final_norm_a), at<T>(e, e->final_norm), at<T>(e, e->final_norm_b), hw, D);
+    CK(cudaGetLastError());
+    e->launches++;
+    TRY((product<T, T, float, EPI_NONE>(e, hw, D, 0, at<T>(e, e->head), D, 1, 0, e->logits, e->cfg.vocab, 0, n_want, e->cfg.vocab, D, 1)));
+    finish_logits(e, n_want);
+    CK(cudaGetLastError());
+  }
+  return 0;
+}
+
 // threads of a row's norm block: about one warp per 256 elements, at least one warp per part while parts <= 32, at most 1024
 static int norm_threads(int D, int G) {
   int nw = std::max(1, std::min(32, D / 256));
@@ -1492,6 +1645,7 @@ static int norm_threads(int D, int G) {
 template <typename T>
 static int run_layers(xotb200_lm* e, const StepPlan& sp, int n_want) {
   if (e->cfg.block == XOTB200_LM_BLOCK_PRE_SCALAR) return run_layers_pre_scalar<T>(e, sp, n_want);
+  if (e->cfg.block == XOTB200_LM_BLOCK_PRE_DYT) return run_layers_pre_dyt<T>(e, sp, n_want);
   if (e->cfg.block != XOTB200_LM_BLOCK_GROUP_RMS) return run_layers_post<T>(e, sp, n_want);
   const int D = e->cfg.width, G = e->cfg.norm_groups, M = sp.M;
   const float eps = e->cfg.norm_eps;
@@ -1569,7 +1723,7 @@ int xotb200_lm_create(const xotb200_lm_cfg* cfg, const xotb200_lm_layer* layers,
   REQUIRE(cfg->width >= 1 && cfg->vocab >= 1, "width and vocab must be positive");
   REQUIRE(cfg->norm_groups >= 1 && cfg->width % cfg->norm_groups == 0, "width %d is not a multiple of norm_groups %d", cfg->width, cfg->norm_groups);
   REQUIRE(cfg->block == XOTB200_LM_BLOCK_GROUP_RMS || cfg->block == XOTB200_LM_BLOCK_POST_LN || cfg->block == XOTB200_LM_BLOCK_POST_RMS ||
-              cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR,
+              cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR || cfg->block == XOTB200_LM_BLOCK_PRE_DYT,
           "unknown block form %d", cfg->block);
   REQUIRE(cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR || (cfg->streams == 0 && cfg->canon_taps == 0 && cfg->residual_mult == 0.f),
           "stream copies, input convolutions and a residual multiplier belong to the pre-norm block with one-number weights");
@@ -1579,7 +1733,9 @@ int xotb200_lm_create(const xotb200_lm_cfg* cfg, const xotb200_lm_layer* layers,
   REQUIRE(cfg->max_positions >= 0, "negative max_positions");
   REQUIRE(cfg->block != XOTB200_LM_BLOCK_GROUP_RMS || (!cfg->pos_sinusoid && !cfg->embed_norm),
           "a computed position vector and a norm on the embedding belong to the other block forms");
-  REQUIRE(cfg->block != XOTB200_LM_BLOCK_PRE_SCALAR || (!cfg->pos_sinusoid && cfg->max_positions == 0), "the one-number pre-norm block form adds no position vector");
+  REQUIRE((cfg->block != XOTB200_LM_BLOCK_PRE_SCALAR && cfg->block != XOTB200_LM_BLOCK_PRE_DYT) || (!cfg->pos_sinusoid && cfg->max_positions == 0),
+          "the one-number and the Dynamic-Tanh pre-norm block forms add no position vector");
+  REQUIRE(cfg->block == XOTB200_LM_BLOCK_PRE_DYT || !cfg->layer_scale, "layer scales belong to the Dynamic-Tanh pre-norm block form");
   REQUIRE(!cfg->embed_norm || cfg->block == XOTB200_LM_BLOCK_POST_RMS || cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR,
           "the norm on the embedding is the RMS norm of the post-RMS or the one-number pre-norm block form");
   REQUIRE(!cfg->pos_sinusoid || cfg->sinusoid_base > 0.f, "the computed position vector needs a positive base");
@@ -1753,6 +1909,8 @@ int xotb200_lm_init_synthetic(xotb200_lm* e, uint64_t seed) {
     else if (ends(".r2")) { mean = 1.f; dev = 0.2f; }
     else if (ends(".b") && d.rows == 1) dev = 0.1f;            // biases of projections and layer norms
     else if (ends(".A_log")) dev = 0.3f;
+    else if (ends(".ls1") || ends(".ls2")) { mean = 0.5f; dev = 0.1f; }
+    else if (ends(".correction")) dev = 0.1f;
     else if (name.find("norm") != std::string::npos) { mean = 1.f; dev = 0.1f; }
     else if (d.rows == 1) dev = 0.5f;                  // biases of the delta-rule gates
     else if (name == "embed") dev = 1.f;
@@ -1940,7 +2098,7 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
   std::vector<int> qpis, windows;
   for (auto& L : e->layers)
     if (L.s.mixer == XOTB200_LM_MIX_LATENT_ATTN) {
-      const int q = std::max(1, 32 / L.s.heads);
+      const int q = latent_rows_per_item(L.s);
       if (std::find(qpis.begin(), qpis.end(), q) == qpis.end()) qpis.push_back(q);
       if (use_flash && std::find(windows.begin(), windows.end(), L.s.window) == windows.end()) windows.push_back(L.s.window);
     } else if (L.s.mixer == XOTB200_LM_MIX_ATTENTION) {
@@ -2052,10 +2210,12 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
   sp.max_len = decode_shape ? cdiv(sp.max_len, 256) * 256 : sp.max_len;
   // the key-run buffer is sized before anything is captured: a captured step must not replace a buffer
   for (auto& L : e->layers)
-    if (L.s.mixer == XOTB200_LM_MIX_ATTENTION) {
+    if (L.s.mixer == XOTB200_LM_MIX_ATTENTION || L.s.mixer == XOTB200_LM_MIX_LATENT_ATTN) {
+      const bool latent = L.s.mixer == XOTB200_LM_MIX_LATENT_ATTN;
       int run = 0;
-      const int splits = gqa_key_runs(e, L.s, item_off[-gqa_rows_per_item(L.s)].second, sp.max_len, &run);
-      const size_t need = splits > 1 ? (size_t)M * L.s.heads * splits * (2 + L.s.vdim) : 0;
+      const int splits = latent ? latent_key_runs(e, L.s, item_off[latent_rows_per_item(L.s)].second, sp.max_len, &run)
+                                : gqa_key_runs(e, L.s, item_off[-gqa_rows_per_item(L.s)].second, sp.max_len, &run);
+      const size_t need = splits > 1 ? (size_t)M * L.s.heads * splits * (2 + (latent ? L.s.kv_rank : L.s.vdim)) : 0;
       if (need > e->part_cap) { drop_graphs(e); TRY(regrow(e->part, need * 4)); e->part_cap = need; }
     }
   GraphSlot* gs = nullptr;

@@ -2,7 +2,8 @@
 // reads the residual stream itself; a layer norm with weight and bias, or an RMS norm with a weight stored around zero, closes it),
 // with a learned position table or a computed sine/cosine position vector, short causal convolutions in front of a gated delta
 // rule, the two-sided xIELU activation and mixtures of experts (gated silu or relu^2 experts, two routing rules).
-// Also the pre-norm block form whose norm weights are one number each: the stream kept in several copies mixed by
+// Also the pre-norm block form with a Dynamic Tanh norm (dyt_rows_kernel and the closing epilogue of layered_kernels.cuh), and the
+// pre-norm block form whose norm weights are one number each: the stream kept in several copies mixed by
 // hyper-connections, and a causal convolution added to every sublayer input (embed_streams_kernel, hc_open_kernel, short_conv_kernel).
 //
 // Number formats as in layered_kernels.cuh: T is the storage type of weights and GEMM inputs (bf16 serving, float in the 32-bit
@@ -137,6 +138,38 @@ __global__ void residual_rmsnorm_kernel(float* __restrict__ x, const float* __re
     }
     if (h) stf(h + (size_t)m * D + d, v);
   }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------
+// Pre-norm block whose norm is a Dynamic Tanh, tanh(alpha x) * w + b (XOTB200_LM_BLOCK_PRE_DYT).  Between two sublayers it is part of the
+// closing epilogue (EPI_CLOSE); these kernels serve the places without a product in front:
+//   embed_dyt_rows_kernel  x = embed[token]                 (fp32), h = dyt(x)
+//   dyt_rows_kernel        h[m] = dyt(x[src_rows[m]])               (the first sublayer of a later shard; the final norm of the wanted rows)
+//   close_rows_kernel      stream_close of a sublayer output y whose last kernel does not close
+// ---------------------------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void embed_dyt_rows_kernel(const T* __restrict__ embed, const int* __restrict__ tokens, const T* __restrict__ alpha, const T* __restrict__ w,
+                                      const T* __restrict__ b, float* __restrict__ x, T* __restrict__ h, int D) {
+  const size_t m = blockIdx.x;
+  const T* src = embed + (size_t)tokens[m] * D;
+  const float a = ldf(alpha);
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    const float v = ldf(src + d);
+    x[m * D + d] = v;
+    stf(h + m * D + d, dyt_f(v, a, ldf(w + d), ldf(b + d)));
+  }
+}
+template <typename T>
+__global__ void dyt_rows_kernel(const float* __restrict__ x, const int* __restrict__ src_rows, const T* __restrict__ alpha, const T* __restrict__ w,
+                                const T* __restrict__ b, T* __restrict__ h, int D) {
+  const size_t m = blockIdx.x, xm = src_rows ? src_rows[m] : m;
+  const float a = ldf(alpha);
+  for (int d = threadIdx.x; d < D; d += blockDim.x) stf(h + m * D + d, dyt_f(x[xm * D + d], a, ldf(w + d), ldf(b + d)));
+}
+template <typename T>
+__global__ void close_rows_kernel(const EpiArgs close, const float* __restrict__ y, int D) {
+  const size_t m = blockIdx.x;
+  for (int d = threadIdx.x; d < D; d += blockDim.x) stream_close<T>(close, m, d, y[m * D + d]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
@@ -343,18 +376,38 @@ __device__ __forceinline__ void row_dot4x2(const T* const (&wa)[4], const T* con
   for (int i = 0; i < 4; ++i) { ra[i] = warp_sum(a[i]); rb[i] = warp_sum(b[i]); }
 }
 
+// index of the largest of v[0 .. n) (shared memory; the lower index on ties), the same on every lane; entries that are NaN or minus
+// infinity are passed over, 0 when nothing is left
+__device__ __forceinline__ int warp_argmax(const float* v, int n, int lane) {
+  float b = -INFINITY;
+  int bi = 0x7fffffff;
+  for (int i = lane; i < n; i += 32)
+    if (v[i] > b) { b = v[i]; bi = i; }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, b, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ob > b || (ob == b && oi < bi)) { b = ob; bi = oi; }
+  }
+  return bi < n ? bi : 0;
+}
+
 // ---------------------------------------------------------------------------------------------------------------------------
 // Mixture of experts, router: logits z = W_r h (+ bias) in fp32 (h in T).
 //   kind 0: scores s = softmax(z) over all E experts; experts form `groups` equal groups of neighbours, a group's score is its best
 //           expert's, only experts of the `keep` best groups can be chosen; the `top` best of those are the token's experts,
 //           weighted by their s (not renormalised);
-//   kind 1: the `top` largest logits are the token's experts, weighted by the softmax over those `top` logits only.
+//   kind 1: the `top` largest logits are the token's experts, weighted by the softmax over those `top` logits only;
+//   kind 2: scores s = sigmoid(z), CHOICE scores c = s + correction (may be negative); a group's score is the sum of its `group_best`
+//           largest c, only experts of the `keep` best groups can be chosen; the `top` largest c of those are the token's experts,
+//           weighted by their s over the sum of the chosen s, times wscale.  The whole warp selects.
 // Ties go to the lower index.  One block per row (its warps share the experts' logits, warp 0 selects); dynamic shared memory:
-// D + E floats.
+// D + E floats (kind 2: D + 2 E + groups).
 // ---------------------------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void moe_router_kernel(const T* __restrict__ h, int D, const T* __restrict__ w_router, const T* __restrict__ bias, int kind, int E,
-                                  int groups, int keep, int top, int* __restrict__ ids, float* __restrict__ wts, int M) {
+                                  int groups, int keep, int top, const T* __restrict__ correction, int group_best, float wscale, int* __restrict__ ids,
+                                  float* __restrict__ wts, int M) {
   extern __shared__ __align__(16) float rsm[];                 // [D] the row (fp32), then [E] scores
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int m = blockIdx.x;
@@ -386,6 +439,48 @@ __global__ void moe_router_kernel(const T* __restrict__ h, int D, const T* __res
       }
       for (int k = 0; k < top; ++k) wts[(size_t)m * top + k] /= den;
     }
+    return;
+  }
+  if (kind == 2) {
+    float *c = s + E, *gs = c + E;                             // choice scores, group scores
+    for (int e = lane; e < E; e += 32) {
+      s[e] = sigmoidf_(s[e]);
+      c[e] = s[e] + (correction ? ldf(correction + e) : 0.f);
+    }
+    __syncwarp();
+    if (groups > 1) {
+      const int per = E / groups;
+      for (int g = lane; g < groups; g += 32) {
+        float b1 = -INFINITY, b2 = -INFINITY;                  // the two largest of the group
+        for (int e = 0; e < per; ++e) {
+          const float v = c[(size_t)g * per + e];
+          if (v > b1) { b2 = b1; b1 = v; }
+          else b2 = fmaxf(b2, v);
+        }
+        gs[g] = group_best == 2 && per > 1 ? b1 + b2 : b1;
+      }
+      __syncwarp();
+      for (int k = 0; k < keep; ++k) {                         // the best group left is kept: its score becomes NaN
+        const int g = warp_argmax(gs, groups, lane);
+        if (lane == 0) gs[g] = __int_as_float(0x7fffffff);
+        __syncwarp();
+      }
+      for (int e = lane; e < E; e += 32)
+        if (gs[e / per] == gs[e / per]) c[e] = -INFINITY;      // not kept
+      __syncwarp();
+    }
+    float sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+      const int e = warp_argmax(c, E, lane);
+      if (lane == 0) {
+        ids[(size_t)m * top + k] = e;
+        wts[(size_t)m * top + k] = s[e];
+        c[e] = -INFINITY;                                      // taken
+      }
+      sum += s[e];
+      __syncwarp();
+    }
+    for (int k = lane; k < top; k += 32) wts[(size_t)m * top + k] = wts[(size_t)m * top + k] / (sum + 1e-20f) * wscale;
     return;
   }
   float mx = -INFINITY;
@@ -428,24 +523,18 @@ __global__ void moe_router_kernel(const T* __restrict__ h, int D, const T* __res
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// Mixture of experts: layout of an expert's gate and up matrices.  w_gu is [E][2 F, D]; with il8 (F a multiple of 8) gate row f
-// and up row f sit at rows (f / 8) * 16 + f % 8 and (f / 8) * 16 + 8 + f % 8, so that a 16-column fragment of a product's output
-// holds 8 gate values next to their 8 up values and silu(gate) * up is formed in the epilogue; else gate rows come first, then up.
-// ---------------------------------------------------------------------------------------------------------------------------
-__device__ __host__ __forceinline__ size_t moe_gate_row(int f, int F, int il8) { return il8 ? (size_t)(f / 8) * 16 + f % 8 : (size_t)f; }
-__device__ __host__ __forceinline__ size_t moe_up_row(int f, int F, int il8) { return il8 ? (size_t)(f / 8) * 16 + 8 + f % 8 : (size_t)F + f; }
-
-// ---------------------------------------------------------------------------------------------------------------------------
 // Mixture of experts, row form (few rows, and the 32-bit mode): every (row, chosen expert) streams that expert's matrices.
-//   moe_rows_up_kernel   act[m, k, f] = silu(W_gate[e] h_m)[f] * (W_up[e] h_m)[f],  e = ids[m, k]        one warp per f
-//                        ungated experts (w_gu is then [E][F, D], up rows only): act[m, k, f] = relu(W_up[e] h_m)[f]^2
+//   moe_rows_up_kernel   act[m, k, f] = glu((W_gate[e] h_m)[f], (W_up[e] h_m)[f]),  e = ids[m, k]        one warp per f
+//                        gated experts (EXPERT_GLU = 1: silu(g) u, 2: the clamped gate of `glu`; rows laid out as glu_gate_row / glu_up_row say)
+//                        ungated experts (EXPERT_GLU = 0; w_gu is then [E][F, D], up rows only): act[m, k, f] = relu(W_up[e] h_m)[f]^2
 //   moe_rows_down_kernel y[m, d] (+)= sum_k wts[m, k] * (W_down[e_k] act[m, k, :])[d]                    one warp per d
 // w_down: [E][D, F].  With `accumulate` the sum is added to what y holds (a shared expert's output made by ordinary products).
 // A shared expert of ungated form can also ride along: w_shared [Fs, D] is one more "expert" of moe_rows_up_kernel (grid y = top,
 // its activations go to act_shared [M, Fs]), and moe_rows_down_kernel adds W_sdown act_shared with weight one (w_sdown [D, Fs]).
+// With close.x the sum is not written to y but closes the sublayer (stream_close).
 // ---------------------------------------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void moe_rows_up_kernel(const T* __restrict__ h, int D, const T* __restrict__ w_gu, int F, int il8, int gated, const int* __restrict__ ids,
+__global__ void moe_rows_up_kernel(const T* __restrict__ h, int D, const T* __restrict__ w_gu, int F, int expert_glu, const EpiArgs glu, const int* __restrict__ ids,
                                    int top, T* __restrict__ act, const T* __restrict__ w_shared, int Fs, T* __restrict__ act_shared) {
   extern __shared__ __align__(16) float hs[];                  // the row, fp32
   const int m = blockIdx.x, k = blockIdx.y;
@@ -453,7 +542,7 @@ __global__ void moe_rows_up_kernel(const T* __restrict__ h, int D, const T* __re
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const bool vec = D % (16 / sizeof(T)) == 0 && (reinterpret_cast<uintptr_t>(w_gu) & 15) == 0 && (reinterpret_cast<uintptr_t>(w_shared) & 15) == 0;
-  if (!gated) {                                                // four up rows per pass: four loads in flight per lane
+  if (!expert_glu) {                                           // four up rows per pass: four loads in flight per lane
     const bool sh = k == top;                                  // the shared expert rides along as grid row `top`
     const T* we = sh ? w_shared : w_gu + (size_t)ids[(size_t)m * top + k] * F * D;
     T* out = sh ? act_shared + (size_t)m * Fs : act + ((size_t)m * top + k) * F;
@@ -477,14 +566,14 @@ __global__ void moe_rows_up_kernel(const T* __restrict__ h, int D, const T* __re
   const T* we = w_gu + (size_t)ids[(size_t)m * top + k] * 2 * F * D;
   for (int f = blockIdx.z * nw + warp; f < F; f += gridDim.z * nw) {
     float g, u;
-    row_dot2(we + moe_gate_row(f, F, il8) * D, we + moe_up_row(f, F, il8) * D, hs, hs, D, lane, vec, g, u);
-    if (lane == 0) stf(act + ((size_t)m * top + k) * F + f, siluf_(g) * u);
+    row_dot2(we + glu_gate_row(f, F, glu.il8) * D, we + glu_up_row(f, F, glu.il8) * D, hs, hs, D, lane, vec, g, u);
+    if (lane == 0) stf(act + ((size_t)m * top + k) * F + f, expert_glu == 2 ? glu_f<EPI_CLAMPED_GLU>(g, u, glu) : glu_f<EPI_SILU_GLU>(g, u, glu));
   }
 }
 template <typename T>
 __global__ void moe_rows_down_kernel(const T* __restrict__ act, int F, const T* __restrict__ w_down, int D, const int* __restrict__ ids,
                                      const float* __restrict__ wts, int top, int accumulate, float* __restrict__ y, const T* __restrict__ act_shared,
-                                     const T* __restrict__ w_sdown, int Fs) {
+                                     const T* __restrict__ w_sdown, int Fs, const EpiArgs close) {
   extern __shared__ __align__(16) float as[];                  // [top][F] fp32, then [Fs] of the shared expert (from a 16-byte boundary)
   const int m = blockIdx.x;
   float* as_s = as + (((size_t)top * F + 3) & ~(size_t)3);
@@ -544,8 +633,17 @@ __global__ void moe_rows_down_kernel(const T* __restrict__ act, int F, const T* 
       out2 += r1;
     }
     if (lane == 0) {
-      y[(size_t)m * D + d] = accumulate ? y[(size_t)m * D + d] + out : out;
-      if (two) y[(size_t)m * D + d2] = accumulate ? y[(size_t)m * D + d2] + out2 : out2;
+      if (accumulate) {
+        out += y[(size_t)m * D + d];
+        if (two) out2 += y[(size_t)m * D + d2];
+      }
+      if (close.x) {
+        stream_close<T>(close, m, d, out);
+        if (two) stream_close<T>(close, m, d2, out2);
+      } else {
+        y[(size_t)m * D + d] = out;
+        if (two) y[(size_t)m * D + d2] = out2;
+      }
     }
   }
 }
@@ -555,7 +653,7 @@ __global__ void moe_rows_down_kernel(const T* __restrict__ act, int F, const T* 
 // run padded to whole 128-row tiles, and two tensor-core products run over the tiles with the expert's matrices chosen per tile.
 //   moe_plan_kernel    (one block)  counts -> padded run starts, tile -> expert map (-1 beyond the last run), cursors reset
 //   moe_scatter_kernel (one warp per pair) takes the pair's place in its expert's run, remembers it, copies the row there
-//   moe_combine_kernel y[m, :] (+)= sum_k wts[m, k] * yg[place[m, k], :]
+//   moe_combine_kernel y[m, :] (+)= sum_k wts[m, k] * yg[place[m, k], :]      (close.x: closes the sublayer instead)
 // ints: counts[E], starts[E + 1], cursor[E], then tile_expert[n_tiles].  The order of pairs inside a run depends on scheduling; a
 // pair's result does not (rows of a product are independent).
 // ---------------------------------------------------------------------------------------------------------------------------
@@ -614,13 +712,16 @@ __global__ void moe_scatter_kernel(const T* __restrict__ h, int D, const int* __
     for (int d = lane; d < D; d += 32) dst[d] = src[d];
   }
 }
+template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ yg, const int* __restrict__ place, const float* __restrict__ wts, int top, int D,
-                                   int accumulate, float* __restrict__ y) {
+                                   int accumulate, float* __restrict__ y, const EpiArgs close) {
   const size_t m = blockIdx.x;
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k) acc = fmaf(wts[m * top + k], yg[(size_t)place[m * top + k] * D + d], acc);
-    y[m * D + d] = accumulate ? y[m * D + d] + acc : acc;
+    if (accumulate) acc += y[m * D + d];
+    if (close.x) stream_close<T>(close, m, d, acc);
+    else y[m * D + d] = acc;
   }
 }
 

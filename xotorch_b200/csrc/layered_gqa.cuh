@@ -57,13 +57,6 @@ __device__ __forceinline__ int gqa_blocks_seen(int pos, int window, int pool) { 
 __device__ __forceinline__ float gqa_query_temperature(float coef, int every, int pos) {
   return coef != 0.f ? 1.0f + coef * logf((float)((pos + 1) / every + 1)) : 1.0f;
 }
-// folds a sink into finished softmax statistics: returns the factor for the accumulator, updates the denominator
-__device__ __forceinline__ float gqa_apply_sink(float sink, float mx, float& den) {
-  const float nmx = fmaxf(mx, sink);
-  const float corr = mx == -INFINITY ? 0.f : expf(mx - nmx);
-  den = den * corr + expf(sink - nmx);
-  return corr;
-}
 
 template <typename T>
 __device__ __forceinline__ float gqa_adjust(float dot, const GqaScore& sc, float r1, float r2, const float* __restrict__ rel_head, int dist) {
@@ -330,7 +323,7 @@ __global__ void gqa_attention_kernel(const float* __restrict__ qf, const T* __re
     }
     return;
   }
-  const float corr = sc.sink ? gqa_apply_sink(ldf(static_cast<const T*>(sc.sink) + h), mx, den) : 1.0f;
+  const float corr = sc.sink ? apply_sink(ldf(static_cast<const T*>(sc.sink) + h), mx, den) : 1.0f;
   const float inv = corr / den;
   T* o = out + (size_t)m * H * dv + (size_t)h * dv;
 #pragma unroll
@@ -567,7 +560,7 @@ gqa_flash_kernel(const bf16* __restrict__ q16, const bf16* __restrict__ pool, Pa
     const int qi = warp * 16 + gq + r * 8;
     if (qi >= tl.n_rows) continue;
     const size_t m = tl.row0 + qi;
-    const float corr = sc.sink ? gqa_apply_sink(__bfloat162float(static_cast<const bf16*>(sc.sink)[h]), mx[r], den[r]) : 1.0f;
+    const float corr = sc.sink ? apply_sink(__bfloat162float(static_cast<const bf16*>(sc.sink)[h]), mx[r], den[r]) : 1.0f;
     const float inv = corr / den[r];
     bf16* dst = out + m * ((size_t)H * dv) + (size_t)h * dv;
 #pragma unroll

@@ -47,6 +47,68 @@ __device__ __forceinline__ float xielu_f(float z, float ap, float aq) {
 // the exact gelu: z (1 + erf(z / sqrt 2)) / 2
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 
+// its tanh form: z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) / 2
+__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.79788456080286536f * fmaf(0.044715f * z * z, z, z))); }
+// clamped gate:  g' sigmoid(slope g') (u' + 1)  with g' = min(g, limit), u' = u clamped to [-limit, limit]
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float slope) {
+  const float gc = fminf(g, limit), uc = fminf(fmaxf(u, -limit), limit);
+  return gc * sigmoidf_(slope * gc) * (uc + 1.0f);
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------
+// Epilogues of the products.  C holds act(A B^T) with
+//   NONE: itself;  RELU2: relu(.)^2;  XIELU (raw parameters at p);  GELU: exact gelu;
+//   *_GLU: B holds gate and up rows of F pairs (glu_gate_row / glu_up_row), C [*, F] receives silu(g) u, gelu_tanh(g) u or the clamped gate;
+//   CLOSE: C is not written.  The product is a sublayer's output y: it closes the sublayer and opens the next,
+//          x += ls * y (fp32 stream; ls NULL = 1),  h = tanh(alpha x) * w + b  (T; h NULL = no sublayer follows).
+//          A pre-norm that needs no statistic of the row makes this possible: every entry of the stream is finished where it is made.
+// ---------------------------------------------------------------------------------------------------------------------------
+enum { EPI_NONE = 0, EPI_RELU2 = 1, EPI_XIELU = 2, EPI_SILU_GLU = 3, EPI_GELU = 4, EPI_CLOSE = 5, EPI_GELU_GLU = 6, EPI_CLAMPED_GLU = 7 };
+__host__ __device__ constexpr bool epi_is_glu(int epi) { return epi == EPI_SILU_GLU || epi == EPI_GELU_GLU || epi == EPI_CLAMPED_GLU; }
+
+struct EpiArgs {
+  const void* p = nullptr;                             // XIELU: its two raw parameters (T)
+  float limit = 0.f, slope = 0.f;                      // CLAMPED_GLU
+  int il8 = 0;                                         // *_GLU: gate and up rows interleaved in eights (else F gate rows, then F up rows)
+  float* x = nullptr;                                  // CLOSE: the stream [*, ld]
+  void* h = nullptr;                                   // CLOSE: the next operand [*, ld] (T)
+  const void *ls = nullptr, *alpha = nullptr, *w = nullptr, *b = nullptr;   // CLOSE: layer scale; the next norm's weights (T)
+  long ld = 0;
+};
+
+// Layout of the gate and up matrices of a gated feed-forward: [2 F, D]; interleaved (F a multiple of 8) gate row f and up row f sit
+// at rows (f / 8) * 16 + f % 8 and (f / 8) * 16 + 8 + f % 8, so that a 16-column fragment of a product's output holds 8 gate values
+// next to their 8 up values and the gate is formed in the epilogue; else the gate rows come first, then the up rows.
+__device__ __host__ __forceinline__ size_t glu_gate_row(int f, int F, int il8) { return il8 ? (size_t)(f / 8) * 16 + f % 8 : (size_t)f; }
+__device__ __host__ __forceinline__ size_t glu_up_row(int f, int F, int il8) { return il8 ? (size_t)(f / 8) * 16 + 8 + f % 8 : (size_t)F + f; }
+
+template <int EPI>
+__device__ __forceinline__ float glu_f(float g, float u, const EpiArgs& a) {
+  if (EPI == EPI_SILU_GLU) return siluf_(g) * u;
+  if (EPI == EPI_GELU_GLU) return gelu_tanh_f(g) * u;
+  return clamped_glu_f(g, u, a.limit, a.slope);
+}
+__device__ __forceinline__ float dyt_f(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+
+// entry (m, n) of a sublayer's output: closes the sublayer, opens the next
+template <typename T>
+__device__ __forceinline__ void stream_close(const EpiArgs& a, size_t m, int n, float y) {
+  const size_t i = m * a.ld + n;
+  const float x = fmaf(y, a.ls ? ldf(static_cast<const T*>(a.ls) + n) : 1.0f, a.x[i]);
+  a.x[i] = x;
+  if (a.h)
+    stf(static_cast<T*>(a.h) + i,
+        dyt_f(x, ldf(static_cast<const T*>(a.alpha)), ldf(static_cast<const T*>(a.w) + n), ldf(static_cast<const T*>(a.b) + n)));
+}
+
+// folds a sink (a score without key or value) into finished softmax statistics: updates the denominator, returns the factor for the accumulator
+__device__ __forceinline__ float apply_sink(float sink, float mx, float& den) {
+  const float nmx = fmaxf(mx, sink);
+  const float corr = mx == -INFINITY ? 0.f : expf(mx - nmx);
+  den = den * corr + expf(sink - nmx);
+  return corr;
+}
+
 // Where a request's token lives in a paged pool: page_table[slot * pages_per_slot + pos / P] * P + pos % P.
 struct Paging {
   const int* page_table;
@@ -151,61 +213,67 @@ __device__ __forceinline__ void rot_pair_index(int i, int dims, int layout, int&
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
-// Latent cache append.  proj[m, col0 : col0 + R + dr] is the down-projection of row m: the first R columns are RMS-normed (weight
-// w_norm) into the latent, the last dr are the shared key part, of which the first rot_dims entries are rotated by the row's
-// position.  Both go to the row's place in the paged pool: pool[(page * P + offset) * (R + dr) + ...].  One warp per row.
+// Everything between a latent-attention layer's projections and its scores, one warp per (row, head) and one more per row:
+//   warp h < H : query head h of row m (qraw [M, ld], dn unrotated + dr rotated entries per head).  The first rot_dims entries of the
+//                rotated part are turned by the row's position.
+//                absorbed form (qn != NULL): unrotated part -> qn[m, h, dn] (T: the operand of the key-absorption product), rotated part
+//                -> qfull[m, h, R : R + dr] (fp32; columns [0, R) are filled by that product);
+//                expanded form (q16 != NULL): both parts -> q16[m, h, dn + dr] (bf16).
+//   warp H     : cache append.  proj[m, col_kv : col_kv + R + dr] is the row's down-projection: the first R columns are RMS-normed
+//                (weight w_norm) into the latent, the last dr are the shared key part, turned like the queries.  Both go to the row's
+//                place in the paged pool, [latent | key part].
 // ---------------------------------------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void latent_append_kernel(const float* __restrict__ proj, int ld, int col0, int R, int dr, const T* __restrict__ w_norm, float eps,
-                                     const float* __restrict__ freqs, int rot_dims, int layout, const int* __restrict__ row_slot,
-                                     const int* __restrict__ row_pos, Paging pg, T* __restrict__ pool, int M) {
-  const int m = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (m >= M) return;
-  const float* r = proj + (size_t)m * ld + col0;
-  T* dst = pool + pg.row(row_slot[m], row_pos[m]) * (size_t)(R + dr);
-  float s = 0.f;
-  for (int d = lane; d < R; d += 32) s = fmaf(r[d], r[d], s);
-  const float rs = 1.0f / sqrtf(warp_sum(s) / (float)R + eps);
-  for (int d = lane; d < R; d += 32) stf(dst + d, r[d] * rs * ldf(w_norm + d));
+__global__ void latent_prepare_kernel(const float* __restrict__ qraw, int q_ld, int H, int dn, int dr, const float* __restrict__ proj, int ld, int col_kv, int R,
+                                      const T* __restrict__ w_norm, float eps, const float* __restrict__ freqs, int rot_dims, int layout,
+                                      const int* __restrict__ row_slot, const int* __restrict__ row_pos, Paging pg, T* __restrict__ pool, T* __restrict__ qn,
+                                      float* __restrict__ qfull, bf16* __restrict__ q16, int M) {
+  const long idx = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (idx >= (long)M * (H + 1)) return;
+  const int m = (int)(idx / (H + 1)), h = (int)(idx % (H + 1));
   const float p = (float)row_pos[m];
-  const float* kr = r + R;
-  for (int i = lane; i < rot_dims / 2; i += 32) {
-    int a, b;
-    rot_pair_index(i, rot_dims, layout, a, b);
-    const float ang = p * freqs[i], c = cosf(ang), sn = sinf(ang);
-    const float u = kr[a], v = kr[b];
-    stf(dst + R + a, u * c - v * sn);
-    stf(dst + R + b, v * c + u * sn);
+  if (h == H) {
+    const float* r = proj + (size_t)m * ld + col_kv;
+    T* dst = pool + pg.row(row_slot[m], row_pos[m]) * (size_t)(R + dr);
+    float s = 0.f;
+    for (int d = lane; d < R; d += 32) s = fmaf(r[d], r[d], s);
+    const float rs = 1.0f / sqrtf(warp_sum(s) / (float)R + eps);
+    for (int d = lane; d < R; d += 32) stf(dst + d, r[d] * rs * ldf(w_norm + d));
+    const float* kr = r + R;
+    for (int i = lane; i < rot_dims / 2; i += 32) {
+      int a, b;
+      rot_pair_index(i, rot_dims, layout, a, b);
+      const float ang = p * freqs[i], c = cosf(ang), sn = sinf(ang);
+      const float u = kr[a], v = kr[b];
+      stf(dst + R + a, u * c - v * sn);
+      stf(dst + R + b, v * c + u * sn);
+    }
+    for (int d = rot_dims + lane; d < dr; d += 32) stf(dst + R + d, kr[d]);
+    return;
   }
-  for (int d = rot_dims + lane; d < dr; d += 32) stf(dst + R + d, kr[d]);
-}
-
-// ---------------------------------------------------------------------------------------------------------------------------
-// Query split.  qraw[m, h * (dn + dr) + ...] (fp32 projection output, leading dimension ld, first column col0) is cut per head
-// into the unrotated part -> qn[m, h, dn] (T: the operand of the key-absorption product) and the rotated part, turned by the
-// row's position -> qfull[m, h, R : R + dr] (fp32; columns [0, R) are filled by the absorption product).  One warp per (row, head).
-// ---------------------------------------------------------------------------------------------------------------------------
-template <typename T>
-__global__ void query_split_kernel(const float* __restrict__ qraw, int ld, int col0, int H, int dn, int dr, int R, const float* __restrict__ freqs,
-                                   int rot_dims, int layout, const int* __restrict__ row_pos, T* __restrict__ qn, float* __restrict__ qfull,
-                                   int M) {
-  const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (idx >= M * H) return;
-  const int m = idx / H, h = idx % H;
-  const float* q = qraw + (size_t)m * ld + col0 + (size_t)h * (dn + dr);
-  for (int d = lane; d < dn; d += 32) stf(qn + ((size_t)m * H + h) * dn + d, q[d]);
-  float* out = qfull + ((size_t)m * H + h) * (R + dr) + R;
-  const float p = (float)row_pos[m];
+  const float* q = qraw + (size_t)m * q_ld + (size_t)h * (dn + dr);
   const float* qr = q + dn;
+  T* on = qn ? qn + ((size_t)m * H + h) * dn : nullptr;
+  float* of = qn ? qfull + ((size_t)m * H + h) * (R + dr) + R : nullptr;
+  bf16* o16 = q16 ? q16 + ((size_t)m * H + h) * (dn + dr) : nullptr;
+  for (int d = lane; d < dn; d += 32) {
+    if (on) stf(on + d, q[d]);
+    if (o16) o16[d] = __float2bfloat16_rn(q[d]);
+  }
+  auto put = [&](int d, float v) {
+    if (of) of[d] = v;
+    if (o16) o16[dn + d] = __float2bfloat16_rn(v);
+  };
   for (int i = lane; i < rot_dims / 2; i += 32) {
     int a, b;
     rot_pair_index(i, rot_dims, layout, a, b);
     const float ang = p * freqs[i], c = cosf(ang), sn = sinf(ang);
     const float u = qr[a], v = qr[b];
-    out[a] = u * c - v * sn;
-    out[b] = v * c + u * sn;
+    put(a, u * c - v * sn);
+    put(b, v * c + u * sn);
   }
-  for (int d = rot_dims + lane; d < dr; d += 32) out[d] = qr[d];
+  for (int d = rot_dims + lane; d < dr; d += 32) put(d, qr[d]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
@@ -217,7 +285,8 @@ __global__ void query_split_kernel(const float* __restrict__ qraw, int ld, int c
 // One CTA serves one work item = up to `q_per_item` consecutive rows of one request, all H heads; one WARP owns one (row, head)
 // pair: lane j scores key j of a 32-key tile held in shared memory (fp32, row stride padded odd), the softmax statistics are
 // exchanged by shuffles, and the lanes then split the R latent columns of the running sum sum_j p_j c_j between them
-// (NACC = ceil(R / 32) registers).  Output: olat[m, h, R] (T), times sigmoid(gate[m, h]) when the mixer has an output gate.
+// (NACC = ceil(R / 32) registers).  Output: olat[m, h, R] (T), times sigmoid(gate[m, h]) when the mixer has an output gate.  With a
+// sink (per head, may be NULL) the softmax denominator also holds exp(sink[h]): a term without key or value, folded in once at the end.
 // ---------------------------------------------------------------------------------------------------------------------------
 struct Item {
   int row0;     // first packed row
@@ -233,7 +302,7 @@ struct Item {
 template <typename T, int NACC>
 __global__ void latent_attention_kernel(const float* __restrict__ qfull, const T* __restrict__ pool, Paging pg, const Item* __restrict__ items,
                                         int H, int R, int dr, float scale, int window, const float* __restrict__ gate, int gate_ld,
-                                        int gate_col0, T* __restrict__ olat, int chunk, float* __restrict__ part) {
+                                        int gate_col0, const T* __restrict__ sink, T* __restrict__ olat, int chunk, float* __restrict__ part) {
   extern __shared__ float smem[];
   const Item it = items[blockIdx.x];
   const int W = R + dr, WS = W | 1;                 // odd row stride: lane j reading row j is conflict-free
@@ -311,7 +380,8 @@ __global__ void latent_attention_kernel(const float* __restrict__ qfull, const T
     }
     return;
   }
-  float g = 1.0f / den;
+  const float corr = sink ? apply_sink(ldf(sink + h), mx, den) : 1.0f;
+  float g = corr / den;
   if (gate) g *= sigmoidf_(gate[(size_t)m * gate_ld + gate_col0 + h]);
   T* out = olat + ((size_t)m * H + h) * R;
 #pragma unroll
@@ -322,10 +392,11 @@ __global__ void latent_attention_kernel(const float* __restrict__ qfull, const T
 }
 
 // merges the key runs of latent_attention_kernel: one warp per (row, head) pair of the listed items (grid.y covers the pairs);
-// lane z first turns run z's {max, sum} into its weight exp(max_z - max) (at most 32 runs), then the lanes split the R columns
+// lane z first turns run z's {max, sum} into its weight exp(max_z - max) (at most 32 runs), then the lanes split the R columns.  A
+// sink joins here, once, like a run that holds the weight exp(sink) and no values.
 template <typename T>
 __global__ void latent_attention_combine_kernel(const float* __restrict__ part, const Item* __restrict__ items, int H, int R, int splits,
-                                                const float* __restrict__ gate, int gate_ld, int gate_col0, T* __restrict__ olat) {
+                                                const float* __restrict__ gate, int gate_ld, int gate_col0, const T* __restrict__ sink, T* __restrict__ olat) {
   const Item it = items[blockIdx.x];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int pair = blockIdx.y * nw + warp;
@@ -333,17 +404,20 @@ __global__ void latent_attention_combine_kernel(const float* __restrict__ part, 
   const int m = it.row0 + pair / H, h = pair % H;
   const float* src = part + ((size_t)m * H + h) * splits * (size_t)(2 + R);
   const float mz = lane < splits ? src[(size_t)lane * (2 + R)] : -INFINITY;
-  const float mx = warp_max(mz);
+  const float sk = sink ? ldf(sink + h) : -INFINITY;
+  const float mx = fmaxf(warp_max(mz), sk);
   const float wz = mz == -INFINITY ? 0.f : expf(mz - mx);
-  const float den = warp_sum(lane < splits ? src[(size_t)lane * (2 + R) + 1] * wz : 0.f);
+  const float den = warp_sum(lane < splits ? src[(size_t)lane * (2 + R) + 1] * wz : 0.f) + (sink ? expf(sk - mx) : 0.f);
   float g = 1.0f / den;
   if (gate) g *= sigmoidf_(gate[(size_t)m * gate_ld + gate_col0 + h]);
   for (int d0 = 0; d0 < R; d0 += 32) {
     const int d = d0 + lane;
     float a = 0.f;
-    for (int z = 0; z < splits; ++z) {
-      const float w = __shfl_sync(0xffffffffu, wz, z);
-      if (w != 0.f && d < R) a = fmaf(src[(size_t)z * (2 + R) + 2 + d], w, a);
+#pragma unroll 8
+    for (int z = 0; z < splits; ++z) {                 // loads without a branch, so that several are in flight: a run that saw no
+      const float w = __shfl_sync(0xffffffffu, wz, z); // key has parked zeros and weighs zero
+      const float v = d < R ? src[(size_t)z * (2 + R) + 2 + d] : 0.f;
+      a = fmaf(v, w, a);
     }
     if (d < R) stf(olat + ((size_t)m * H + h) * R + d, a * g);
   }
@@ -545,13 +619,13 @@ __global__ void tanh_cols_kernel(const float* __restrict__ in, int ld, int col0,
 // ---------------------------------------------------------------------------------------------------------------------------
 // Products.  C[z][m, n] = sum_k A[z][m, k] * B[z][n, k]   with fp32 accumulation; A row-major (lda), B addressed by two strides
 // (sbn, sbk) so that a weight stored [K, N] is used without a transposed copy, z = batch (per-head products) via element offsets.
-// EPI 1: C = relu(C)^2.  EPI 2: C = xIELU(C) with the two raw parameters p, q at `epi` (in the weights' type).  EPI 4: C = gelu(C), exact.
+// EPI: see EpiArgs.  With a gated epilogue N counts weight rows (2 F) and virtual row v is the gate (v even) or up (v odd) row of pair v / 2.
 // gemm_tiled_kernel: 64 x 64 x 16 shared-memory tiles, 256 threads, 4 x 4 outputs per thread, fp32 FMA (exact fp32 in the 32-bit mode).
 // ---------------------------------------------------------------------------------------------------------------------------
 template <typename TA, typename TB, typename TC, int EPI>
 __global__ void __launch_bounds__(256)
 gemm_tiled_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __restrict__ B, long sbn, long sbk, long b_batch, TC* __restrict__ C,
-                  long ldc, long c_batch, int M, int N, int K, const TB* __restrict__ epi) {
+                  long ldc, long c_batch, int M, int N, int K, const EpiArgs epi) {
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float As[BK][BM + 4], Bs[BK][BN + 4];
   A += (size_t)blockIdx.z * a_batch;
@@ -568,7 +642,9 @@ gemm_tiled_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __
     if (sbk == 1) {
       for (int e = threadIdx.x; e < BN * BK; e += 256) {
         const int r = e / BK, k = e % BK;
-        Bs[k][r] = (n0 + r < N && k0 + k < K) ? ldf(B + (size_t)(n0 + r) * sbn + k0 + k) : 0.f;
+        size_t row = n0 + r;
+        if constexpr (epi_is_glu(EPI)) row = (n0 + r) & 1 ? glu_up_row((n0 + r) >> 1, N >> 1, epi.il8) : glu_gate_row((n0 + r) >> 1, N >> 1, epi.il8);
+        Bs[k][r] = (n0 + r < N && k0 + k < K) ? ldf(B + row * sbn + k0 + k) : 0.f;
       }
     } else {
       for (int e = threadIdx.x; e < BN * BK; e += 256) {
@@ -592,7 +668,7 @@ gemm_tiled_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __
     __syncthreads();
   }
   float ap = 0.f, aq = 0.f;
-  if (EPI == 2) { ap = softplusf_(ldf(epi)); aq = 0.5f + softplusf_(ldf(epi + 1)); }
+  if (EPI == EPI_XIELU) { ap = softplusf_(ldf(static_cast<const TB*>(epi.p))); aq = 0.5f + softplusf_(ldf(static_cast<const TB*>(epi.p) + 1)); }
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -600,10 +676,16 @@ gemm_tiled_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (m < M && n < N) {
         float v = acc[i][j];
-        if (EPI == 1) { v = fmaxf(v, 0.f); v *= v; }
-        if (EPI == 2) v = xielu_f(v, ap, aq);
-        if (EPI == 4) v = gelu_erf_f(v);
-        stf(C + (size_t)m * ldc + n, v);
+        if constexpr (epi_is_glu(EPI)) {
+          if (j % 2 == 0) stf(C + (size_t)m * ldc + n / 2, glu_f<EPI>(v, acc[i][j + 1 < 4 ? j + 1 : j], epi));
+        } else if constexpr (EPI == EPI_CLOSE) {
+          stream_close<TB>(epi, m, n, v);
+        } else {
+          if (EPI == EPI_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+          if (EPI == EPI_XIELU) v = xielu_f(v, ap, aq);
+          if (EPI == EPI_GELU) v = gelu_erf_f(v);
+          stf(C + (size_t)m * ldc + n, v);
+        }
       }
     }
 }
@@ -615,7 +697,7 @@ gemm_tiled_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __
 template <typename TA, typename TB, typename TC, int EPI, int MR>
 __global__ void __launch_bounds__(256)
 gemv_rows_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __restrict__ B, long sbn, long b_batch, TC* __restrict__ C, long ldc,
-                 long c_batch, int M, int N, int K, int wsplit, const TB* __restrict__ epi) {
+                 long c_batch, int M, int N, int K, int wsplit, const EpiArgs epi) {
   constexpr int RB = 4;
   extern __shared__ float a_s[];                     // [M][K], then the slice sums [8 warps][RB][MR]
   A += (size_t)blockIdx.z * a_batch;
@@ -634,6 +716,12 @@ gemv_rows_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __r
   const int kbeg = slice * ksl, kend = min(K, kbeg + ksl);
   for (int nb = blockIdx.x * gpb * RB; nb < N; nb += gridDim.x * gpb * RB) {   // uniform trip count for the whole block
     const int n0 = nb + grp * RB;
+    size_t brow[RB];                                 // element offset of the group's weight rows
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      brow[r] = (size_t)(n0 + r) * sbn;
+      if constexpr (epi_is_glu(EPI)) brow[r] = (r & 1 ? glu_up_row((n0 + r) >> 1, N >> 1, epi.il8) : glu_gate_row((n0 + r) >> 1, N >> 1, epi.il8)) * (size_t)sbn;
+    }
     float acc[RB][MR];
 #pragma unroll
     for (int r = 0; r < RB; ++r)
@@ -647,7 +735,7 @@ gemv_rows_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __r
         for (int u = 0; u < 2; ++u)
 #pragma unroll
           for (int r = 0; r < RB; ++r)
-            raw[u][r] = (n0 + r < N && k + u * 32 * VEC < kend) ? *reinterpret_cast<const uint4*>(B + (size_t)(n0 + r) * sbn + k + u * 32 * VEC)
+            raw[u][r] = (n0 + r < N && k + u * 32 * VEC < kend) ? *reinterpret_cast<const uint4*>(B + brow[r] + k + u * 32 * VEC)
                                                                 : make_uint4(0, 0, 0, 0);
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
@@ -670,7 +758,7 @@ gemv_rows_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __r
       for (int k = kbeg + lane; k < kend; k += 32) {
 #pragma unroll
         for (int r = 0; r < RB; ++r) {
-          const float w = n0 + r < N ? ldf(B + (size_t)(n0 + r) * sbn + k) : 0.f;
+          const float w = n0 + r < N ? ldf(B + brow[r] + k) : 0.f;
 #pragma unroll
           for (int m = 0; m < MR; ++m)
             if (m < M) acc[r][m] = fmaf(a_s[m * K + k], w, acc[r][m]);
@@ -690,10 +778,20 @@ gemv_rows_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __r
       float v = 0.f;
       for (int sidx = 0; sidx < wsplit; ++sidx) v += red[((warp + sidx) * RB + r) * MR + m];   // fixed order: deterministic
       if (m < M && n0 + r < N) {
-        if (EPI == 1) { v = fmaxf(v, 0.f); v *= v; }
-        if (EPI == 2) v = xielu_f(v, softplusf_(ldf(epi)), 0.5f + softplusf_(ldf(epi + 1)));
-        if (EPI == 4) v = gelu_erf_f(v);
-        stf(C + (size_t)m * ldc + n0 + r, v);
+        if constexpr (epi_is_glu(EPI)) {
+          if (r % 2 == 0) {
+            float u = 0.f;                           // the up row's sum: r + 1
+            for (int sidx = 0; sidx < wsplit; ++sidx) u += red[((warp + sidx) * RB + r + 1) * MR + m];
+            stf(C + (size_t)m * ldc + (n0 + r) / 2, glu_f<EPI>(v, u, epi));
+          }
+        } else if constexpr (EPI == EPI_CLOSE) {
+          stream_close<TB>(epi, m, n0 + r, v);
+        } else {
+          if (EPI == EPI_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+          if (EPI == EPI_XIELU) v = xielu_f(v, softplusf_(ldf(static_cast<const TB*>(epi.p))), 0.5f + softplusf_(ldf(static_cast<const TB*>(epi.p) + 1)));
+          if (EPI == EPI_GELU) v = gelu_erf_f(v);
+          stf(C + (size_t)m * ldc + n0 + r, v);
+        }
       }
     }
     __syncthreads();
@@ -796,7 +894,8 @@ __global__ void copy_rows_f32_kernel(const float* __restrict__ src, float* __res
 // per (64-row tile, head) with mma.sync.m16n8k16 (bf16 operands, fp32 accumulators): scores = [q_unrot | q_rot] . [kn | kr],
 // fp32 scale / mask / running max and sum, and the weights enter the value product as a bf16 PAIR (high part + remainder, two
 // MMAs) so that they keep 16 mantissa bits instead of 8.  Key range as in the absorbed kernel: j <= i and (window == 0 or
-// i - j < window).  Output: o[m, h * dv + :] (bf16), times sigmoid(gate[m, h]) when the mixer is gated.
+// i - j < window).  Output: o[m, h * dv + :] (bf16), times sigmoid(gate[m, h]) when the mixer is gated; a sink joins the finished
+// statistics of a row (apply_sink).
 // ===========================================================================================================================
 constexpr int FLASH_MIN_ROWS = 16;
 
@@ -825,28 +924,6 @@ __global__ void latent_gather_kernel(const T* __restrict__ pool, Paging pg, cons
   for (int d = lane; d < W; d += 32) dst[d] = src[d];
 }
 
-// Query in 16 bits for the expanded form: q16[m, h, 0:dn] = unrotated part, q16[m, h, dn:dn+dr] = rotated part turned by the position
-__global__ void query_rotate16_kernel(const float* __restrict__ qraw, int ld, int H, int dn, int dr, const float* __restrict__ freqs, int rot_dims,
-                                      int layout, const int* __restrict__ row_pos, bf16* __restrict__ q16, int M) {
-  const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (idx >= M * H) return;
-  const int m = idx / H, h = idx % H;
-  const float* q = qraw + (size_t)m * ld + (size_t)h * (dn + dr);
-  bf16* out = q16 + ((size_t)m * H + h) * (dn + dr);
-  for (int d = lane; d < dn; d += 32) out[d] = __float2bfloat16_rn(q[d]);
-  const float p = (float)row_pos[m];
-  const float* qr = q + dn;
-  for (int i = lane; i < rot_dims / 2; i += 32) {
-    int a, b;
-    rot_pair_index(i, rot_dims, layout, a, b);
-    const float ang = p * freqs[i], c = cosf(ang), sn = sinf(ang);
-    const float u = qr[a], v = qr[b];
-    out[dn + a] = __float2bfloat16_rn(u * c - v * sn);
-    out[dn + b] = __float2bfloat16_rn(v * c + u * sn);
-  }
-  for (int d = rot_dims + lane; d < dr; d += 32) out[dn + d] = __float2bfloat16_rn(qr[d]);
-}
-
 __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
@@ -870,7 +947,7 @@ template <int DVT>   // value columns held per warp row: DVT tiles of 8 (dv <= 8
 __global__ void __launch_bounds__(128)
 latent_flash_kernel(const bf16* __restrict__ q16, const bf16* __restrict__ kn, const bf16* __restrict__ cbuf, const bf16* __restrict__ vx,
                     const FlashTile* __restrict__ tiles, int H, int dn, int dr, int dv, int R, float scale, int window, const float* __restrict__ gate,
-                    int gate_ld, int gate_col0, bf16* __restrict__ out) {
+                    int gate_ld, int gate_col0, const bf16* __restrict__ sink, bf16* __restrict__ out) {
   extern __shared__ __align__(16) uint8_t fsm[];
   const FlashTile tl = tiles[blockIdx.x];
   const int h = blockIdx.y;
@@ -1001,7 +1078,8 @@ latent_flash_kernel(const bf16* __restrict__ q16, const bf16* __restrict__ kn, c
     const int qi = warp * 16 + g + r * 8;
     if (qi >= tl.n_rows) continue;
     const int m = tl.row0 + qi;
-    float sc = 1.0f / den[r];
+    const float corr = sink ? apply_sink(__bfloat162float(sink[h]), mx[r], den[r]) : 1.0f;
+    float sc = corr / den[r];
     if (gate) sc *= sigmoidf_(gate[(size_t)m * gate_ld + gate_col0 + h]);
     bf16* dst = out + (size_t)m * ((size_t)H * dv) + (size_t)h * dv;
 #pragma unroll
@@ -1033,7 +1111,7 @@ template <int DVT>
 __global__ void __launch_bounds__(128)
 latent_flash_aligned_kernel(const bf16* __restrict__ q16, const bf16* __restrict__ kn, const bf16* __restrict__ cbuf, const bf16* __restrict__ vx,
                             const FlashTile* __restrict__ tiles, int H, int dn, int dr, int dv, int R, float scale, int window,
-                            const float* __restrict__ gate, int gate_ld, int gate_col0, bf16* __restrict__ out) {
+                            const float* __restrict__ gate, int gate_ld, int gate_col0, const bf16* __restrict__ sink, bf16* __restrict__ out) {
   extern __shared__ __align__(16) uint8_t fsm[];
   const FlashTile tl = tiles[blockIdx.x];
   const int h = blockIdx.y;
@@ -1170,7 +1248,8 @@ latent_flash_aligned_kernel(const bf16* __restrict__ q16, const bf16* __restrict
     const int qi = warp * 16 + g + r * 8;
     if (qi >= tl.n_rows) continue;
     const int m = tl.row0 + qi;
-    float sc = 1.0f / den[r];
+    const float corr = sink ? apply_sink(__bfloat162float(sink[h]), mx[r], den[r]) : 1.0f;
+    float sc = corr / den[r];
     if (gate) sc *= sigmoidf_(gate[(size_t)m * gate_ld + gate_col0 + h]);
     bf16* dst = out + (size_t)m * ((size_t)H * dv) + (size_t)h * dv;
 #pragma unroll

@@ -6,8 +6,8 @@
 // (cp.async.bulk.tensor.3d, SWIZZLE_128B; coordinates {k, row, batch}), a single thread issues tcgen05.mma.cta_group::1.kind::f16
 // into a tensor-memory accumulator, four warps read it back with tcgen05.ld and store it (fp32 or bf16, optionally relu(.)^2).
 // Rows beyond M, columns beyond N and the tail of K come from the tensor map's zero fill, so no size has to be a multiple of the
-// tile.  EPI 1: relu(.)^2; EPI 2: xIELU; EPI 4: exact gelu; EPI 3: the columns come in groups of 16 = 8 gate values followed by their 8 up values, and
-// C [*, N / 2] receives silu(gate) * up.  With `tile_batch` every row tile takes its B matrix from a list (grouped products: rows
+// tile.  EPI: see EpiArgs (layered_kernels.cuh); gated epilogues: the columns come in groups of 16 = 8 gate values followed by their 8 up values, and
+// C [*, N / 2] receives the gated value.  With `tile_batch` every row tile takes its B matrix from a list (grouped products: rows
 // sorted by expert).  The PTX wrappers are those of the shard engine's prefill GEMM (prefill_tc.cuh); what differs is the operand layout
 // (plain row-major weights, batched per-head products through the third coordinate), the epilogue and that EVERY wait is bounded:
 // a wait that expires sets *err and the CTA drains, frees its tensor memory and returns.
@@ -39,7 +39,7 @@ struct LtcArgs {
   void* C;          // fp32 or bf16 [*, ldc]
   long ldc, c_batch;
   int* err;
-  const __nv_bfloat16* epi;   // EPI 2: the two raw xIELU parameters
+  EpiArgs epi;
   const int* tile_batch;      // not NULL: row tile t reads B's batch tile_batch[t] (A and C are not batched); a negative entry = the tile is empty
   int cols_first;             // 1: blockIdx.x walks the column tiles and blockIdx.y the row tiles (CTAs that run together share few row tiles:
                               // a grouped product then streams an expert's matrix while only that expert's rows are in flight)
@@ -49,6 +49,12 @@ template <typename TC>
 __device__ __forceinline__ void ltc_store(TC* p, float v);
 template <> __device__ __forceinline__ void ltc_store<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void ltc_store<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// 16 consecutive bf16 (from a 16-byte boundary)
+__device__ __forceinline__ void ltc_load16(__nv_bfloat16* dst, const __nv_bfloat16* src) {
+  reinterpret_cast<uint4*>(dst)[0] = reinterpret_cast<const uint4*>(src)[0];
+  reinterpret_cast<uint4*>(dst)[1] = reinterpret_cast<const uint4*>(src)[1];
+}
 
 template <int NT, int EPI, int NS, typename TC>
 __global__ void __launch_bounds__(LTC_THREADS, 2 * ltc_smem_bytes(NT, NS) <= 226 * 1024 ? 2 : 1)
@@ -123,7 +129,14 @@ ltc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
       const bool vec = (sizeof(TC) == 4) && ((a.ldc | a.c_batch) % 4 == 0) && ((reinterpret_cast<uintptr_t>(a.C) & 15) == 0);
       const bool vec16 = (sizeof(TC) == 2) && ((a.ldc | a.c_batch) % 8 == 0) && ((reinterpret_cast<uintptr_t>(a.C) & 15) == 0);
       float ap = 0.f, aq = 0.f;
-      if (EPI == 2) { ap = softplusf_(__bfloat162float(a.epi[0])); aq = 0.5f + softplusf_(__bfloat162float(a.epi[1])); }
+      if (EPI == EPI_XIELU) {
+        const __nv_bfloat16* raw = static_cast<const __nv_bfloat16*>(a.epi.p);
+        ap = softplusf_(__bfloat162float(raw[0]));
+        aq = 0.5f + softplusf_(__bfloat162float(raw[1]));
+      }
+      // CLOSE: whole 16-entry pieces of the stream row, its operand row and the per-entry vectors move in 16-byte accesses
+      const bool vecx = EPI == EPI_CLOSE && a.epi.ld % 8 == 0;
+      const float alpha = EPI == EPI_CLOSE && a.epi.h ? __bfloat162float(*static_cast<const __nv_bfloat16*>(a.epi.alpha)) : 0.f;
 #pragma unroll 1
       for (int c0 = 0; c0 < NT; c0 += 16) {
         uint32_t v[16];
@@ -131,10 +144,49 @@ ltc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
         const int n = n0 + c0;
         if (row >= a.M || n >= a.N) continue;
         float f[16];
-        if constexpr (EPI == 3) {                      // 8 gate values, then their 8 up values -> 8 outputs at columns n / 2 ..
+        if constexpr (EPI == EPI_CLOSE) {
+          if (vecx && n + 16 <= a.N) {
+            float4* x4 = reinterpret_cast<float4*>(a.epi.x + (size_t)row * a.epi.ld + n);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              const float4 t = x4[j];
+              f[4 * j] = t.x; f[4 * j + 1] = t.y; f[4 * j + 2] = t.z; f[4 * j + 3] = t.w;
+            }
+            __align__(16) __nv_bfloat16 t[16];
+            if (a.epi.ls) {
+              ltc_load16(t, static_cast<const __nv_bfloat16*>(a.epi.ls) + n);
+#pragma unroll
+              for (int j = 0; j < 16; ++j) f[j] = fmaf(__uint_as_float(v[j]), __bfloat162float(t[j]), f[j]);
+            } else {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) f[j] += __uint_as_float(v[j]);
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) x4[j] = make_float4(f[4 * j], f[4 * j + 1], f[4 * j + 2], f[4 * j + 3]);
+            if (a.epi.h) {
+              __align__(16) __nv_bfloat16 tb[16];
+              ltc_load16(t, static_cast<const __nv_bfloat16*>(a.epi.w) + n);
+              ltc_load16(tb, static_cast<const __nv_bfloat16*>(a.epi.b) + n);
+              uint32_t pk[8];
+#pragma unroll
+              for (int j = 0; j < 8; ++j) {
+                __nv_bfloat162 h2 = __floats2bfloat162_rn(dyt_f(f[2 * j], alpha, __bfloat162float(t[2 * j]), __bfloat162float(tb[2 * j])),
+                                                          dyt_f(f[2 * j + 1], alpha, __bfloat162float(t[2 * j + 1]), __bfloat162float(tb[2 * j + 1])));
+                pk[j] = *reinterpret_cast<uint32_t*>(&h2);
+              }
+              uint4* d4 = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.epi.h) + (size_t)row * a.epi.ld + n);
+              d4[0] = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+              d4[1] = make_uint4(pk[4], pk[5], pk[6], pk[7]);
+            }
+          } else {
+#pragma unroll 1
+            for (int j = 0; j < 16; ++j)
+              if (n + j < a.N) stream_close<__nv_bfloat16>(a.epi, row, n + j, __uint_as_float(v[j]));
+          }
+        } else if constexpr (epi_is_glu(EPI)) {        // 8 gate values, then their 8 up values -> 8 outputs at columns n / 2 ..
           const int no = n >> 1;
 #pragma unroll
-          for (int j = 0; j < 8; ++j) f[j] = siluf_(__uint_as_float(v[j])) * __uint_as_float(v[j + 8]);
+          for (int j = 0; j < 8; ++j) f[j] = glu_f<EPI>(__uint_as_float(v[j]), __uint_as_float(v[j + 8]), a.epi);
           if (sizeof(TC) == 2 && a.ldc % 8 == 0 && (reinterpret_cast<uintptr_t>(a.C) & 15) == 0) {
             uint32_t pk[4];
 #pragma unroll
@@ -151,9 +203,9 @@ ltc_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           f[j] = __uint_as_float(v[j]);
-          if (EPI == 1) { f[j] = fmaxf(f[j], 0.f); f[j] *= f[j]; }
-          if (EPI == 2) f[j] = xielu_f(f[j], ap, aq);
-          if (EPI == 4) f[j] = gelu_erf_f(f[j]);
+          if (EPI == EPI_RELU2) { f[j] = fmaxf(f[j], 0.f); f[j] *= f[j]; }
+          if (EPI == EPI_XIELU) f[j] = xielu_f(f[j], ap, aq);
+          if (EPI == EPI_GELU) f[j] = gelu_erf_f(f[j]);
         }
         if (vec && n + 16 <= a.N) {
           float4* d4 = reinterpret_cast<float4*>(reinterpret_cast<float*>(crow) + n);

@@ -84,6 +84,12 @@ class LayerSpec:
   par_gate_cap: float = 0.0
   mix_scale: float = 1.0
   par_scale: float = 0.0
+  weights_of: int = -1
+  expert_limit: float = 0.0
+  expert_slope: float = 0.0
+  router_correction: int = 0
+  group_best: int = 0
+  router_scale: float = 0.0
 
   def to_c(self) -> LmLayer:
     c = LmLayer()
@@ -318,8 +324,69 @@ def fubelorn_globals(config: dict) -> dict:
               canon_taps=int((config.get("canon") or {}).get("taps", 0)), residual_mult=float(config.get("residual_mult", 1.0)))
 
 
+# ---- the Rinutar family ------------------------------------------------------------------------------------------------------
+# config.json: {"architecture": "Rinutar", "width", "vocab", "norm": {"eps"}, "layers": [{"type", "mixer", "mlp", "weights_of"?}]}
+# A layer is pre-norm with a Dynamic Tanh and a layer scale: x += ls1 * mixer(tanh(alpha x) * w + b), x += ls2 * ff(...); the logits use the
+# embedding table.  norm.eps belongs to the norm of the latents.
+#   type "latent_attention"  direct queries, pairs (i, i + dims/2) of the rotated part turned, causal, one sink logit per head in the
+#                            softmax denominator, no gate (mixer: heads, dim, rot_dim, vdim, kv_rank, rot {base, dims}, scale)
+#   mlp.kind "dense"         W_down (gelu_tanh(W_gate h) * W_up h) (mlp.ff)
+#   mlp.kind "moe"           clamped gated experts (mlp.expert {ff, limit}); sigmoid scores, corrected for the choice, groups scored by their two
+#                            best (mlp.router {experts, top, groups {count, keep}, scale})
+#   weights_of: j            the layer uses layer j's tensors, with a cache of its own
+RINUTAR_GLU_SLOPE, RINUTAR_GROUP_BEST = 1.702, 2
+
+
+def _rinutar_ff(i: int, mlp) -> dict:
+  if mlp is None:
+    return dict(ff=0, ff_kind=_lib.LM_FF_GELU_GATED)
+  kind = mlp.get("kind", "dense")
+  if kind == "dense":
+    return dict(ff=int(mlp["ff"]), ff_kind=_lib.LM_FF_GELU_GATED)
+  if kind == "moe":
+    r, e = mlp["router"], mlp["expert"]
+    groups = r.get("groups") or {}
+    count = int(groups.get("count", 1))
+    return dict(ff=0, ff_kind=_lib.LM_FF_MOE, experts=int(r["experts"]), top=int(r["top"]), expert_ff=int(e["ff"]), groups=count,
+                groups_keep=int(groups.get("keep", count)), expert_act=_lib.LM_EXPERT_CLAMPED_GLU, expert_limit=float(e["limit"]),
+                expert_slope=RINUTAR_GLU_SLOPE, router_kind=_lib.LM_ROUTER_SIGMOID_GROUPS, router_correction=1, group_best=RINUTAR_GROUP_BEST,
+                router_scale=float(r["scale"]))
+  raise ValueError(f"layer {i}: feed-forward kind {kind!r} is not implemented (dense, moe)")
+
+
+def weight_owner(layers: List[dict], i: int) -> int:
+  """the layer whose tensors layer i uses: `weights_of` followed to a layer that has its own"""
+  seen = {i}
+  while layers[i].get("weights_of") is not None:
+    i = int(layers[i]["weights_of"])
+    if i in seen or not 0 <= i < len(layers):
+      raise ValueError(f"weights_of leads to layer {i}, which has no tensors of its own")
+    seen.add(i)
+  return i
+
+
+def rinutar_layers(config: dict, shapes: Dict[str, Tuple[int, ...]]) -> List[LayerSpec]:
+  out, layers = [], config["layers"]
+  for i, layer in enumerate(layers):
+    kind, m = layer["type"], layer["mixer"]
+    if kind != "latent_attention":
+      raise ValueError(f"layer {i}: mixer type {kind!r} is not implemented")
+    rot, src = m.get("rot") or {}, weight_owner(layers, i)
+    out.append(LayerSpec(
+      mixer=_lib.LM_MIX_LATENT_ATTN, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), rot_dim=int(m["rot_dim"]), kv_rank=int(m["kv_rank"]),
+      rot_dims=int(rot.get("dims", m["rot_dim"])), rot_layout=_lib.LM_ROT_HALF, rot_base=float(rot.get("base", 10000.0)), scale=float(m["scale"]), sink=1,
+      weights_of=src if src != i else -1, **_rinutar_ff(i, layer.get("mlp"))))
+  return out
+
+
+def rinutar_globals(config: dict) -> dict:
+  return dict(width=int(config["width"]), vocab=int(config["vocab"]), norm_groups=1, norm_eps=float(config["norm"]["eps"]),
+              block=_lib.LM_BLOCK_PRE_DYT, layer_scale=1, tied_head=1)
+
+
 LAYERED_FAMILIES = {"Zokuvik": (zokuvik_layers, zokuvik_globals), "Bufulorn": (bufulorn_layers, bufulorn_globals),
-                    "Tunavik": (tunavik_layers, tunavik_globals), "Fubelorn": (fubelorn_layers, fubelorn_globals)}
+                    "Tunavik": (tunavik_layers, tunavik_globals), "Fubelorn": (fubelorn_layers, fubelorn_globals),
+                    "Rinutar": (rinutar_layers, rinutar_globals)}
 
 
 class LayeredShard:
@@ -379,6 +446,7 @@ class LayeredShard:
     cfg.logit_scale, cfg.logit_softcap = self.globals.get("logit_scale", 1.0), self.globals.get("logit_softcap", 0.0)
     cfg.streams, cfg.canon_taps = self.globals.get("streams", 0), self.globals.get("canon_taps", 0)
     cfg.residual_mult = self.globals.get("residual_mult", 0.0)
+    cfg.layer_scale, cfg.tied_head = self.globals.get("layer_scale", 0), self.globals.get("tied_head", 0)
     cfg.dtype = _lib.LM_DTYPE_F32 if self.dtype == "float32" else _lib.LM_DTYPE_BF16
     arr = (LmLayer * len(specs))(*[s.to_c() for s in specs])
     h = C.c_void_p()
