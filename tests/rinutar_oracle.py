@@ -186,7 +186,7 @@ def random_weights(cfg: dict, seed: int) -> Dict[str, Tensor]:
     elif last in ("ls1", "ls2"):
       t = rnd(shape, 0.6, 0.2)
     elif last == "correction":
-      t = rnd(shape, -0.7, 0.4)                       # most choice scores are negative
+      t = rnd(shape, -0.9, 0.6)                       # most choice scores are negative
     elif last == "b":
       t = rnd(shape, 0.0, 0.2)
     elif "norm" in last:

@@ -48,7 +48,7 @@ def oracle_logits(cfg, weights, tokens, dtype=torch.float64):
   return lg.double().numpy(), [t.double().numpy() for t in trail]
 
 
-def settled_rows(cfg, weights, tokens, dtype: str, gap=0.03) -> np.ndarray:
+def settled_rows(cfg, weights, tokens, dtype: str, gap=0.015) -> np.ndarray:
   """[T] bool: the rows a test holds to the tolerance.  float32: all.  bfloat16: those where no router choice (an expert over the best
   one left out, a group over the best one dropped) leads by less than `gap`; with the router's input rounded to 16 bits the others may
   legitimately choose otherwise."""

@@ -252,12 +252,15 @@ def test_freed_pages_and_slots_are_clean_for_the_next_request():
 
 
 # ---- keys and sinks made to stand out ----------------------------------------------------------------------------------------
-def plant(cfg, W, boost=6.0):
+def plant(cfg, W):
   """The last token of the vocabulary gets an embedding whose queries are the keys of the last but one: the first norm and the query
-  projection are inverted for it (the rotated query part is aimed at zero, so that the distance does not matter).  Returns (key token,
-  query token)."""
+  projection are inverted for it (the rotated query part is aimed at zero, so that the distance does not matter).  The other
+  tokens' embeddings are small: their own queries stay dull whatever the score scale.  Returns (key token, query token)."""
   m, V = cfg["layers"][0]["mixer"], cfg["vocab"]
   H, dn, dr, R = m["heads"], m["dim"], m["rot_dim"], m["kv_rank"]
+  W["embed"][:V - 2] *= 0.25
+  W["l0.norm1.b"] *= 0.25
+  W["l0.mix.o"] *= 4.0
   D64 = {k: v.double() for k, v in W.items()}
   alpha, w, b = D64["l0.norm1.alpha"], D64["l0.norm1"], D64["l0.norm1.b"]
   hk = ro.dyt(D64["embed"][V - 2], alpha, w, b)
@@ -285,7 +288,7 @@ def test_far_keys_and_page_borders(decode, dtype):
   one by one when `decode`."""
   V, n_tok = 40, 150
   for name, pos, page in (("far", 3, 16), ("first", 0, 16), ("page_first", 64, 64), ("page_last", 63, 64), ("second_token", 1, 8), ("last_page_full", 143, 16), ("newest_but_one", 148, 8)):
-    cfg = config([attn(heads=2, dim=12, rot_dim=4, vdim=12, kv_rank=24, scale=2.0)], vocab=V, width=64)
+    cfg = config([attn(heads=2, dim=12, rot_dim=4, vdim=12, kv_rank=24, scale=12.0)], vocab=V, width=64)
     W = ro.random_weights(cfg, 17)
     key_tok, query_tok = plant(cfg, W)
     seq = rand_tokens(V - 2, n_tok, 5)
@@ -310,8 +313,9 @@ def test_sinks_of_every_size(dtype):
   cfg = config([attn(heads=3, vdim=8, scale=0.1)], width=32)
   W = ro.random_weights(cfg, 29)
   W["l0.mix.sink"] = torch.tensor([9.0, -9.0, 4.5])
+  W["l0.mix.o"] *= 4.0
   toks = rand_tokens(cfg["vocab"], 200, 7)
-  for wrong in (torch.full((3,), -80.0), torch.tensor([9.0, -9.0, 4.5]) * 0.1, torch.tensor([9.0, -9.0, 4.5]) + 1.1):
+  for wrong in (torch.full((3,), -80.0), torch.tensor([9.0, -9.0, 4.5]) * 0.1, torch.tensor([9.0, -9.0, 1.0])):
     other = dict(W)
     other["l0.mix.sink"] = wrong
     assert row_err(oracle_logits(cfg, other, toks)[0], oracle_logits(cfg, W, toks)[0]) > 2 * TOL["bfloat16"], "the sinks must matter"
@@ -342,10 +346,12 @@ def test_choice_scores_and_weights_are_different_things(dtype):
   is negative, so a dropped group that counted as zero would win"""
   cfg = config([attn(mlp=moe(8, 3, 12, (4, 2), 2.0))])
   W = ro.random_weights(cfg, 8)
-  W["l0.mlp.correction"] = torch.tensor([-9.0, -3.0, -7.0, -5.0, -3.5, -8.0, -4.0, -6.0])
+  W["l0.mlp.correction"] = torch.tensor([-19.0, -3.0, -17.0, -5.0, -5.0, -8.0, -6.5, -11.0])
   toks = rand_tokens(cfg["vocab"], 30, 2)
-  ids, _ = ro.route(torch.randn(5, 48, dtype=torch.float64), ro.sub({k: v.double() for k, v in W.items()}, "l0.mlp."), cfg["layers"][0]["mlp"]["router"])
-  assert all(set(r) == {6, 7, 4} for r in ids.tolist()) or all(set(r) == {1, 4, 6} or len(set(r)) == 3 for r in ids.tolist())
+  W["l0.mlp.router"] *= 0.5
+  # groups (-19, -3) (-17, -5) (-5, -8) (-6.5, -11), each plus scores in 0..1: the last two are kept, of them 4, 6 and 5 chosen
+  ids, w = ro.route(torch.randn(50, 48, dtype=torch.float64, generator=torch.Generator().manual_seed(1)), ro.sub({k: v.double() for k, v in W.items()}, "l0.mlp."), cfg["layers"][0]["mlp"]["router"])
+  assert all(set(row) == {4, 5, 6} for row in ids.tolist()) and (w.std(-1) > 0.003).all()
   n = make_engine(cfg, W, dtype)
   check(n, cfg, W, toks, [30], dtype, slot=0)
   check(n, cfg, W, toks, [11, 2, 1], dtype, slot=1)

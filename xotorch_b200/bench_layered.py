@@ -15,6 +15,11 @@ LSTM, windowed attention that keeps the first tokens + gated delta rule; state-s
 stream, input convolutions, gelu feed-forwards) beside the closest existing family on the same engine, a Bufulorn model of gated-delta
 and attention layers with dense feed-forwards, of the same width and depth and (to a few per cent) weight bytes.
 
+`--layered-family rinutar`: the same for Rinutar-shaped models (latent attention with sinks, Dynamic-Tanh blocks, gated gelu feed-forwards and
+clamped gated experts in turn) beside the two closest existing families on the same engine: a Zokuvik model with the same latent attention and
+dense feed-forwards (as many weight bytes as a Rinutar token touches), and a Bufulorn model with the same alternation of dense and expert
+feed-forwards (to a few per cent the same weight bytes).
+
 Timing: every number is the device time of the step(s) (CUDA events on the engine's stream, `last_step_ms` / the ring's own
 timer), after warm-up; the weights of every size are larger than L2 from `medium` on, and each prompt step streams all of them.
 Roofline denominators come from MEASURED_PEAKS.json (fallback: the profiling recipe's numbers)."""
@@ -172,6 +177,36 @@ def bufulorn_dense_config(s: dict, b: dict, context: int, ff: int):
   return {"architecture": "Bufulorn", "width": s["width"], "vocab": s["vocab"], "max_positions": context, "norm": {"eps": 1e-5}, "layers": layers}
 
 
+# Rinutar shapes at the same widths: latent attention heads / ranks as the Zokuvik layers above, six layers with dense gated gelu and
+# expert feed-forwards in turn (16 clamped gated experts of a quarter of the dense inner size, 4 per token, 8 groups of which 4 are kept)
+def rinutar_config(s: dict):
+  mixer = {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot_dim"], "vdim": s["vdim"], "kv_rank": s["kv_rank"],
+           "rot": {"base": 500000.0, "dims": s["rot_dim"]}, "scale": float((s["dim"] + s["rot_dim"]) ** -0.5)}
+  dense = {"kind": "dense", "ff": s["ff"]}
+  moe = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP, "groups": {"count": GROUPS, "keep": KEEP}, "scale": 2.0}, "expert": {"ff": s["ff"] // 4, "limit": 7.0}}
+  layers = [{"type": "latent_attention", "mixer": mixer, "mlp": mlp} for _ in range(3 * s["repeats"] // 2) for mlp in (dense, moe)]
+  cfg = {"architecture": "Rinutar", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "layers": layers}
+  return cfg, len(layers) // 2 * (EXPERTS - TOP) * 3 * (s["ff"] // 4) * s["width"] * 2
+
+
+def zokuvik_attention_config(s: dict):
+  """Zokuvik layers with the same latent attention (direct queries, a window no prompt reaches) and relu^2 feed-forwards of the same bytes"""
+  m = {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot_dim"], "vdim": s["vdim"], "kv_rank": s["kv_rank"], "rot": {"base": 500000.0, "dims": s["rot_dim"]},
+       "scale": float((s["dim"] + s["rot_dim"]) ** -0.5), "mask": {"size": 1 << 20}}
+  layers = [{"type": "latent_attention_2", "mixer": m, "mlp": {"kind": "dense", "ff": s["ff"] * 3 // 2}} for _ in range(3 * s["repeats"])]
+  return {"architecture": "Zokuvik", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6, "groups": 4}, "layers": layers}
+
+
+def bufulorn_alternating_config(s: dict, b: dict, context: int):
+  """Bufulorn attention layers whose feed-forwards are dense (xIELU, two matrices of the bytes of Rinutar's three) and experts in turn"""
+  m = {"heads": b["heads"], "kv_heads": b["kv_heads"], "dim": b["dim"], "vdim": b["vdim"], "scale": float(b["dim"] ** -0.5), "softcap": 30.0}
+  dense = {"kind": "dense", "ff": s["ff"] * 3 // 2}
+  moe = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP, "groups": {"count": GROUPS, "keep": KEEP}}, "expert": {"ff": s["ff"] // 4}}
+  layers = [{"type": "attention", "mixer": m, "mlp": mlp} for _ in range(3 * s["repeats"] // 2) for mlp in (dense, moe)]
+  cfg = {"architecture": "Bufulorn", "width": s["width"], "vocab": s["vocab"], "max_positions": context, "norm": {"eps": 1e-5}, "layers": layers}
+  return cfg, len(layers) // 2 * (EXPERTS - TOP) * 3 * (s["ff"] // 4) * s["width"] * 2
+
+
 def peaks():
   p = ROOT / "MEASURED_PEAKS.json"
   if p.exists():
@@ -193,7 +228,8 @@ def layered_numbers(s: dict, prompts, decode_ctx: int, decode_batches, steps: in
   eng.init_synthetic(7)
   wbytes = eng.weight_bytes()
   # a prompt step streams the body once + one row of the embedding (and of the position table) per token
-  body = wbytes - 2 * s["vocab"] * s["width"] - int(cfg.get("max_positions", 0)) * s["width"] * 2 - idle_bytes
+  tables = 1 if eng.globals.get("tied_head") else 2                      # embedding and head
+  body = wbytes - tables * 2 * s["vocab"] * s["width"] - int(cfg.get("max_positions", 0)) * s["width"] * 2 - idle_bytes
   rng = np.random.default_rng(0)
   out = {"weight_bytes": wbytes, "prefill": {}, "decode": {}}
   max_b = max(decode_batches)
@@ -361,6 +397,22 @@ def run_fubelorn(args, sizes, prompts, hbm, tf, src) -> None:
     print(json.dumps(line), flush=True)
 
 
+def run_rinutar(args, sizes, prompts, hbm, tf, src) -> None:
+  for name in sizes:
+    s, b = SIZES[name], BUFULORN[name]
+    warm = max(3, args.warmup)
+    context = max(max(prompts), 1024 + 9 * (args.steps * 8 + warm)) + 64
+    cfg, idle = rinutar_config(s)
+    bcfg, bidle = bufulorn_alternating_config(s, b, context)
+    models = {"rinutar": (cfg, idle), "zokuvik_active_size": (zokuvik_attention_config(s), 0), "bufulorn_same_size": (bcfg, bidle)}
+    out = {k: layered_numbers(s, prompts, decode_ctx=1024, decode_batches=[1, 8], steps=args.steps, warmup=warm, cfg=c, idle_bytes=i) for k, (c, i) in models.items()}
+    line = {"bench": "layered", "family": "rinutar", "size": name, "dtype": "bf16", "data": "synthetic", "shape": dict(s, **b), "idle_expert_bytes": idle, **out,
+            "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
+            "frac_of_peak": {**{f"{k}_decode1_hbm": round(v["decode"]["1"]["gbs_weights_device"] / hbm, 3) for k, v in out.items()},
+                             **{f"{k}_prefill{n}_tensor": round(v["prefill"][str(n)]["tflops_weights"] / tf, 3) for k, v in out.items() for n in prompts}}}
+    print(json.dumps(line), flush=True)
+
+
 def run(args) -> None:
   hbm, tf, src = peaks()
   sizes = [x for x in (args.layered_sizes or "small,medium,large").split(",") if x]
@@ -371,6 +423,8 @@ def run(args) -> None:
     return run_tunavik(args, sizes, prompts, hbm, tf, src)
   if getattr(args, "layered_family", "") == "fubelorn":
     return run_fubelorn(args, sizes, prompts, hbm, tf, src)
+  if getattr(args, "layered_family", "") == "rinutar":
+    return run_rinutar(args, sizes, prompts, hbm, tf, src)
   for name in sizes:
     s = SIZES[name]
     z = layered_numbers(s, prompts, decode_ctx=1024, decode_batches=[1, 8], steps=args.steps, warmup=max(3, args.warmup))

@@ -949,7 +949,8 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
     const auto& it = sp.items.at(qpi);
     if (it.second > 0) {
       const int pairs = qpi * H, nw = latent_item_warps(s, pairs);
-      const size_t smem = ((size_t)32 * ((R + dr) | 1) + (size_t)nw * (R + dr)) * 4;
+      const int nbuf = latent_smem_bytes<T>(R + dr, nw, 2) <= 200 * 1024 ? 2 : 1;
+      const size_t smem = latent_smem_bytes<T>(R + dr, nw, nbuf);
       int chunk = 0;
       const int splits = latent_key_runs(e, s, it.second, sp.max_len, &chunk);
       REQUIRE(splits == 1 || (size_t)M * H * splits * (2 + R) <= e->part_cap, "internal: the key-run buffer was not sized for this step");
@@ -959,7 +960,7 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
     auto kern = latent_attention_kernel<T, NACC>;                                                                                               \
     TRY(opt_in_smem(kern, smem));                                                                                                               \
     kern<<<grid, nw * 32, smem, e->stream>>>(e->qfull, static_cast<const T*>(L.pool), pg, it.first, H, R, dr, s.scale, s.window, gate, L.n_in, \
-                                             L.c_g, sink, static_cast<T*>(e->olat), chunk, e->part);                                            \
+                                             L.c_g, sink, static_cast<T*>(e->olat), chunk, e->part, nbuf);                                      \
   } while (0)
       if (R <= 64) LAUNCH_ATTN(2);
       else if (R <= 128) LAUNCH_ATTN(4);
@@ -969,7 +970,7 @@ static int attention_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
       CK(cudaGetLastError());
       e->launches++;
       if (splits > 1) {
-        latent_attention_combine_kernel<T><<<dim3(it.second, cdiv(pairs, 8)), 256, 0, e->stream>>>(e->part, it.first, H, R, splits, gate, L.n_in, L.c_g, sink, static_cast<T*>(e->olat));
+        latent_attention_combine_kernel<T><<<dim3(it.second, cdiv(pairs, 8), it.second * cdiv(pairs, 8) < e->sm_count ? std::min(16, cdiv(R, 32)) : 1), 256, 0, e->stream>>>(e->part, it.first, H, R, splits, gate, L.n_in, L.c_g, sink, static_cast<T*>(e->olat));
         CK(cudaGetLastError());
         e->launches++;
       }
@@ -1299,6 +1300,9 @@ static int grouped_product(xotb200_lm* e, const bf16* A, long lda, const bf16* B
 // on decode batches: from 4 rows on the grouped form is faster (each chosen expert is streamed once, however many rows chose it).
 static const int MOE_GROUPED_MIN_ROWS = 3;
 
+// grid of an elementwise kernel over [M, D]: one block per row, a row cut over grid.y while that leaves SMs without a block
+static dim3 row_grid(const xotb200_lm* e, int M, int D, int threads) { return dim3(M, std::max(1, std::min(cdiv(D, threads), e->sm_count / std::max(1, M)))); }
+
 static bool layer_has_ff(const xotb200_lm_layer& s) { return s.ff_kind == XOTB200_LM_FF_MOE ? s.experts > 0 : s.ff > 0; }
 
 // the feed-forward of a layer: h (T) -> y (fp32)
@@ -1330,7 +1334,7 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
       auto kern = moe_router_kernel<T>;
       const size_t rsm = ((size_t)((D + 3) & ~3) + (s.router_kind == XOTB200_LM_ROUTER_SIGMOID_GROUPS ? 2 * E + std::max(1, s.groups) : E)) * 4;
       TRY(opt_in_smem(kern, rsm));
-      kern<<<M, std::min(1024, std::max(64, cdiv(E, 2) * 32)), rsm, e->stream>>>(h, D, at<T>(e, L.router), s.router_bias ? at<T>(e, L.router_b) : nullptr,
+      kern<<<M, std::min(1024, std::max(64, (M <= 16 ? E : cdiv(E, 2)) * 32)), rsm, e->stream>>>(h, D, at<T>(e, L.router), s.router_bias ? at<T>(e, L.router_b) : nullptr,
                                                                                  s.router_kind, E, s.groups, s.groups_keep, top, s.router_correction ? at<T>(e, L.correction) : nullptr,
                                                                                  s.group_best, s.router_scale, e->moe_ids, e->moe_wts, M);
     }
@@ -1357,7 +1361,7 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
         if (r == 1) r = grouped_product<EPI_NONE, float>(e, ma, F, at<bf16>(e, L.w_edown), F, (long)D * F, E, e->moe_yg, D, m_pad, D, F, tile_expert);
         if (r < 0) return r;
         if (r == 1) {
-          moe_combine_kernel<bf16><<<M, 256, 0, e->stream>>>(e->moe_yg, place, e->moe_wts, top, D, shared, e->y, close);
+          moe_combine_kernel<bf16><<<row_grid(e, M, D, 256), 256, 0, e->stream>>>(e->moe_yg, place, e->moe_wts, top, D, shared, e->y, close);
           CK(cudaGetLastError());
           e->launches++;
           e->closed = e->close != nullptr;
@@ -1585,8 +1589,8 @@ static int run_layers_pre_dyt(xotb200_lm* e, const StepPlan& sp, int n_want) {
   T* h = static_cast<T*>(e->h);
   const int nt = std::min(256, std::max(32, cdiv(D, 32) * 32));
   LmLayer& L0 = e->layers.front();
-  if (e->first) embed_dyt_rows_kernel<T><<<M, nt, 0, e->stream>>>(at<T>(e, e->embed), sp.tokens, at<T>(e, L0.norm1a), at<T>(e, L0.norm1), at<T>(e, L0.norm1b), e->x, h, D);
-  else dyt_rows_kernel<T><<<M, nt, 0, e->stream>>>(e->x, nullptr, at<T>(e, L0.norm1a), at<T>(e, L0.norm1), at<T>(e, L0.norm1b), h, D);
+  if (e->first) embed_dyt_rows_kernel<T><<<row_grid(e, M, D, nt), nt, 0, e->stream>>>(at<T>(e, e->embed), sp.tokens, at<T>(e, L0.norm1a), at<T>(e, L0.norm1), at<T>(e, L0.norm1b), e->x, h, D);
+  else dyt_rows_kernel<T><<<row_grid(e, M, D, nt), nt, 0, e->stream>>>(e->x, nullptr, at<T>(e, L0.norm1a), at<T>(e, L0.norm1), at<T>(e, L0.norm1b), h, D);
   CK(cudaGetLastError());
   e->launches++;
   // runs one sublayer: `ls` scales its result; the norm that follows it (a = NULL: none) makes the next operand
@@ -1608,7 +1612,7 @@ static int run_layers_pre_dyt(xotb200_lm* e, const StepPlan& sp, int n_want) {
     e->close = nullptr;
     if (rc < 0) return rc;
     if (!e->closed) {
-      close_rows_kernel<T><<<M, nt, 0, e->stream>>>(close, e->y, D);
+      close_rows_kernel<T><<<row_grid(e, M, D, nt), nt, 0, e->stream>>>(close, e->y, D);
       CK(cudaGetLastError());
       e->launches++;
     }
@@ -1625,7 +1629,7 @@ static int run_layers_pre_dyt(xotb200_lm* e, const StepPlan& sp, int n_want) {
   if (e->trace) e->trace_floats = e->layers.size() * (size_t)M * D;
   if (e->last && n_want > 0) {
     T* hw = static_cast<T*>(e->hw);
-    dyt_rows_kernel<T><<<n_want, nt, 0, e->stream>>>(e->x, sp.want, at<T>(e, e->final_norm_a), at<T>(e, e->final_norm), at<T>(e, e->final_norm_b), hw, D);
+    dyt_rows_kernel<T><<<row_grid(e, n_want, D, nt), nt, 0, e->stream>>>(e->x, sp.want, at<T>(e, e->final_norm_a), at<T>(e, e->final_norm), at<T>(e, e->final_norm_b), hw, D);
     CK(cudaGetLastError());
     e->launches++;
     TRY((product<T, T, float, EPI_NONE>(e, hw, D, 0, at<T>(e, e->head), D, 1, 0, e->logits, e->cfg.vocab, 0, n_want, e->cfg.vocab, D, 1)));

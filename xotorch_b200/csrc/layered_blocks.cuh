@@ -146,6 +146,7 @@ __global__ void residual_rmsnorm_kernel(float* __restrict__ x, const float* __re
 //   embed_dyt_rows_kernel  x = embed[token]                 (fp32), h = dyt(x)
 //   dyt_rows_kernel        h[m] = dyt(x[src_rows[m]])               (the first sublayer of a later shard; the final norm of the wanted rows)
 //   close_rows_kernel      stream_close of a sublayer output y whose last kernel does not close
+// No entry needs another, so with few rows a row is cut over grid.y.
 // ---------------------------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_dyt_rows_kernel(const T* __restrict__ embed, const int* __restrict__ tokens, const T* __restrict__ alpha, const T* __restrict__ w,
@@ -153,7 +154,7 @@ __global__ void embed_dyt_rows_kernel(const T* __restrict__ embed, const int* __
   const size_t m = blockIdx.x;
   const T* src = embed + (size_t)tokens[m] * D;
   const float a = ldf(alpha);
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < D; d += gridDim.y * blockDim.x) {
     const float v = ldf(src + d);
     x[m * D + d] = v;
     stf(h + m * D + d, dyt_f(v, a, ldf(w + d), ldf(b + d)));
@@ -164,12 +165,12 @@ __global__ void dyt_rows_kernel(const float* __restrict__ x, const int* __restri
                                 const T* __restrict__ b, T* __restrict__ h, int D) {
   const size_t m = blockIdx.x, xm = src_rows ? src_rows[m] : m;
   const float a = ldf(alpha);
-  for (int d = threadIdx.x; d < D; d += blockDim.x) stf(h + m * D + d, dyt_f(x[xm * D + d], a, ldf(w + d), ldf(b + d)));
+  for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < D; d += gridDim.y * blockDim.x) stf(h + m * D + d, dyt_f(x[xm * D + d], a, ldf(w + d), ldf(b + d)));
 }
 template <typename T>
 __global__ void close_rows_kernel(const EpiArgs close, const float* __restrict__ y, int D) {
   const size_t m = blockIdx.x;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) stream_close<T>(close, m, d, y[m * D + d]);
+  for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < D; d += gridDim.y * blockDim.x) stream_close<T>(close, m, d, y[m * D + d]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------------
@@ -267,17 +268,30 @@ __global__ void gated_delta_prepare_kernel(const float* __restrict__ cv, int C, 
   }
 }
 
-// dot product of a weight row (T, global) with a row held in shared memory (fp32), 16 bytes per lane per load when `vec`
+// acc += w . x over the 16 bytes of weights in `raw` (T) and as many fp32 values of x (shared memory, on a 16-byte boundary)
+template <typename T>
+__device__ __forceinline__ void dot16(float& acc, const uint4& raw, const float* __restrict__ x) {
+  constexpr int VEC = 16 / sizeof(T);
+  const T* w = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+  for (int v = 0; v < VEC; v += 4) {
+    const float4 xv = *reinterpret_cast<const float4*>(x + v);
+    acc = fmaf(ldf(w + v), xv.x, acc);
+    acc = fmaf(ldf(w + v + 1), xv.y, acc);
+    acc = fmaf(ldf(w + v + 2), xv.z, acc);
+    acc = fmaf(ldf(w + v + 3), xv.w, acc);
+  }
+}
+
+// dot product of a weight row (T, global) with a row held in shared memory (fp32), 16 bytes per lane per load when `vec` (which also says
+// that the row in shared memory is on a 16-byte boundary)
 template <typename T>
 __device__ __forceinline__ float row_dot(const T* __restrict__ w, const float* __restrict__ xs, int n, int lane, bool vec) {
   constexpr int VEC = 16 / sizeof(T);
   float acc = 0.f;
   if (vec) {
-    for (int k = lane * VEC; k < n; k += 32 * VEC) {
-      const uint4 raw = *reinterpret_cast<const uint4*>(w + k);
-#pragma unroll
-      for (int v = 0; v < VEC; ++v) acc = fmaf(ldf(reinterpret_cast<const T*>(&raw) + v), xs[k + v], acc);
-    }
+#pragma unroll 4
+    for (int k = lane * VEC; k < n; k += 32 * VEC) dot16<T>(acc, *reinterpret_cast<const uint4*>(w + k), xs + k);
   } else {
     for (int k = lane; k < n; k += 32) acc = fmaf(ldf(w + k), xs[k], acc);
   }
@@ -297,13 +311,10 @@ __device__ __forceinline__ void row_dot2(const T* __restrict__ w0, const T* __re
       const uint4 p0 = *reinterpret_cast<const uint4*>(w0 + k), p1 = *reinterpret_cast<const uint4*>(w1 + k);
       const uint4 q0 = k2 < n ? *reinterpret_cast<const uint4*>(w0 + k2) : z, q1 = k2 < n ? *reinterpret_cast<const uint4*>(w1 + k2) : z;
       const int kk = k2 < n ? k2 : k;                  // past the end the weights read as zero; the index stays inside x
-#pragma unroll
-      for (int v = 0; v < VEC; ++v) {
-        a0 = fmaf(ldf(reinterpret_cast<const T*>(&p0) + v), x0[k + v], a0);
-        a1 = fmaf(ldf(reinterpret_cast<const T*>(&p1) + v), x1[k + v], a1);
-        a0 = fmaf(ldf(reinterpret_cast<const T*>(&q0) + v), x0[kk + v], a0);
-        a1 = fmaf(ldf(reinterpret_cast<const T*>(&q1) + v), x1[kk + v], a1);
-      }
+      dot16<T>(a0, p0, x0 + k);
+      dot16<T>(a1, p1, x1 + k);
+      dot16<T>(a0, q0, x0 + kk);
+      dot16<T>(a1, q1, x1 + kk);
     }
   } else {
     for (int k = lane; k < n; k += 32) { a0 = fmaf(ldf(w0 + k), x0[k], a0); a1 = fmaf(ldf(w1 + k), x1[k], a1); }
@@ -323,9 +334,7 @@ __device__ __forceinline__ void row_dot4(const T* const (&w)[4], const float* co
 #pragma unroll
       for (int i = 0; i < 4; ++i) p[i] = *reinterpret_cast<const uint4*>(w[i] + k);
 #pragma unroll
-      for (int v = 0; v < VEC; ++v)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) a[i] = fmaf(ldf(reinterpret_cast<const T*>(&p[i]) + v), x[i][k + v], a[i]);
+      for (int i = 0; i < 4; ++i) dot16<T>(a[i], p[i], x[i] + k);
     }
   } else {
     for (int k = lane; k < n; k += 32)
@@ -357,15 +366,12 @@ __device__ __forceinline__ void row_dot4x2(const T* const (&wa)[4], const T* con
         q2[i] = more ? *reinterpret_cast<const uint4*>(wb[i] + k2) : z;
       }
 #pragma unroll
-      for (int v = 0; v < VEC; ++v)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float xv = x[i][k + v], xw = x[i][kk + v];
-          a[i] = fmaf(ldf(reinterpret_cast<const T*>(&p[i]) + v), xv, a[i]);
-          b[i] = fmaf(ldf(reinterpret_cast<const T*>(&q[i]) + v), xv, b[i]);
-          a[i] = fmaf(ldf(reinterpret_cast<const T*>(&p2[i]) + v), xw, a[i]);
-          b[i] = fmaf(ldf(reinterpret_cast<const T*>(&q2[i]) + v), xw, b[i]);
-        }
+      for (int i = 0; i < 4; ++i) {
+        dot16<T>(a[i], p[i], x[i] + k);
+        dot16<T>(b[i], q[i], x[i] + k);
+        dot16<T>(a[i], p2[i], x[i] + kk);
+        dot16<T>(b[i], q2[i], x[i] + kk);
+      }
     }
   } else {
     for (int k = lane; k < n; k += 32)
@@ -413,7 +419,7 @@ __global__ void moe_router_kernel(const T* __restrict__ h, int D, const T* __res
   const int m = blockIdx.x;
   float* hs = rsm;
   float* s = rsm + ((D + 3) & ~3);
-  for (int d = threadIdx.x; d < D; d += blockDim.x) hs[d] = ldf(h + (size_t)m * D + d);
+  stage_f32(hs, h + (size_t)m * D, D);
   __syncthreads();
   const bool vec = D % (16 / sizeof(T)) == 0 && (reinterpret_cast<uintptr_t>(w_router) & 15) == 0;
   for (int e = warp; e < E; e += nw) {                         // the warps share the experts; logits in fp32
@@ -538,7 +544,7 @@ __global__ void moe_rows_up_kernel(const T* __restrict__ h, int D, const T* __re
                                    int top, T* __restrict__ act, const T* __restrict__ w_shared, int Fs, T* __restrict__ act_shared) {
   extern __shared__ __align__(16) float hs[];                  // the row, fp32
   const int m = blockIdx.x, k = blockIdx.y;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) hs[d] = ldf(h + (size_t)m * D + d);
+  stage_f32(hs, h + (size_t)m * D, D);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const bool vec = D % (16 / sizeof(T)) == 0 && (reinterpret_cast<uintptr_t>(w_gu) & 15) == 0 && (reinterpret_cast<uintptr_t>(w_shared) & 15) == 0;
@@ -577,9 +583,8 @@ __global__ void moe_rows_down_kernel(const T* __restrict__ act, int F, const T* 
   extern __shared__ __align__(16) float as[];                  // [top][F] fp32, then [Fs] of the shared expert (from a 16-byte boundary)
   const int m = blockIdx.x;
   float* as_s = as + (((size_t)top * F + 3) & ~(size_t)3);
-  for (int i = threadIdx.x; i < top * F; i += blockDim.x) as[i] = ldf(act + (size_t)m * top * F + i);
-  if (w_sdown)
-    for (int i = threadIdx.x; i < Fs; i += blockDim.x) as_s[i] = ldf(act_shared + (size_t)m * Fs + i);
+  stage_f32(as, act + (size_t)m * top * F, top * F);
+  if (w_sdown) stage_f32(as_s, act_shared + (size_t)m * Fs, Fs);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const bool vec = F % (16 / sizeof(T)) == 0 && (reinterpret_cast<uintptr_t>(w_down) & 15) == 0;
@@ -716,7 +721,7 @@ template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ yg, const int* __restrict__ place, const float* __restrict__ wts, int top, int D,
                                    int accumulate, float* __restrict__ y, const EpiArgs close) {
   const size_t m = blockIdx.x;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < D; d += gridDim.y * blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k) acc = fmaf(wts[m * top + k], yg[(size_t)place[m * top + k] * D + d], acc);
     if (accumulate) acc += y[m * D + d];

@@ -109,6 +109,30 @@ __device__ __forceinline__ float apply_sink(float sink, float mx, float& den) {
   return corr;
 }
 
+__device__ __forceinline__ void cp_async4(float* dst_smem, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst_smem)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst_smem, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst_smem)), "l"(src) : "memory");
+}
+
+// n values of T (global) -> fp32 (shared memory), by the whole block; 16 bytes per load when both sides allow
+template <typename T>
+__device__ __forceinline__ void stage_f32(float* __restrict__ dst, const T* __restrict__ src, int n) {
+  constexpr int VEC = 16 / sizeof(T);
+  if (n % VEC == 0 && ((reinterpret_cast<uintptr_t>(src) | (uintptr_t)__cvta_generic_to_shared(dst)) & 15) == 0) {
+#pragma unroll 4
+    for (int i = threadIdx.x * VEC; i < n; i += blockDim.x * VEC) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(src + i);
+      const T* t = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+      for (int v = 0; v < VEC; v += 4) *reinterpret_cast<float4*>(dst + i + v) = make_float4(ldf(t + v), ldf(t + v + 1), ldf(t + v + 2), ldf(t + v + 3));
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = ldf(src + i);
+  }
+}
+
 // Where a request's token lives in a paged pool: page_table[slot * pages_per_slot + pos / P] * P + pos % P.
 struct Paging {
   const int* page_table;
@@ -283,10 +307,11 @@ __global__ void latent_prepare_kernel(const float* __restrict__ qraw, int q_ld, 
 // ever expanded or stored.  Key range of a query at position i: max(0, i - window + 1) .. i (window == 0: 0 .. i).
 //
 // One CTA serves one work item = up to `q_per_item` consecutive rows of one request, all H heads; one WARP owns one (row, head)
-// pair: lane j scores key j of a 32-key tile held in shared memory (fp32, row stride padded odd), the softmax statistics are
-// exchanged by shuffles, and the lanes then split the R latent columns of the running sum sum_j p_j c_j between them
-// (NACC = ceil(R / 32) registers).  Output: olat[m, h, R] (T), times sigmoid(gate[m, h]) when the mixer has an output gate.  With a
-// sink (per head, may be NULL) the softmax denominator also holds exp(sink[h]): a term without key or value, folded in once at the end.
+// pair: lane j scores key j of a 32-key tile held in shared memory as stored (32-bit words, an odd number of them per row; the next
+// tile arrives by cp.async meanwhile), the softmax statistics are exchanged by shuffles, and the lanes then split the R latent columns
+// of the running sum sum_j p_j c_j between them (NACC registers, NACC >= R / 32).  Output: olat[m, h, R] (T), times
+// sigmoid(gate[m, h]) when the mixer has an output gate.  With a sink (per head, may be NULL) the softmax denominator also holds
+// exp(sink[h]): a term without key or value, folded in once at the end.
 // ---------------------------------------------------------------------------------------------------------------------------
 struct Item {
   int row0;     // first packed row
@@ -299,75 +324,116 @@ struct Item {
 // run z and parks its unnormalised result {running max, sum, accumulator[R]} in `part` ([M * H][gridDim.z][2 + R] fp32), and
 // latent_attention_combine_kernel merges the runs.  That is what keeps a single decoded row over a long context from running on
 // one SM.  With gridDim.z == 1 the kernel normalises, gates and stores itself.
+// shared memory: `nbuf` key tiles of 32 rows of latent_row_words 32-bit words, then one query (fp32, zero-padded to fours) per warp
+template <typename T> __host__ __device__ constexpr int latent_row_words(int W) { return ((W * (int)sizeof(T) + 3) / 4) | 1; }
+template <typename T> __host__ __device__ constexpr size_t latent_smem_bytes(int W, int warps, int nbuf) {
+  return ((size_t)nbuf * 32 * latent_row_words<T>(W) + (size_t)warps * ((W + 3) & ~3)) * 4;
+}
+template <typename T> __device__ __forceinline__ void word_values(uint32_t w, float* v);
+template <> __device__ __forceinline__ void word_values<float>(uint32_t w, float* v) { v[0] = __uint_as_float(w); }
+template <> __device__ __forceinline__ void word_values<bf16>(uint32_t w, float* v) { v[0] = __uint_as_float(w << 16); v[1] = __uint_as_float(w & 0xffff0000u); }
+
 template <typename T, int NACC>
-__global__ void latent_attention_kernel(const float* __restrict__ qfull, const T* __restrict__ pool, Paging pg, const Item* __restrict__ items,
-                                        int H, int R, int dr, float scale, int window, const float* __restrict__ gate, int gate_ld,
-                                        int gate_col0, const T* __restrict__ sink, T* __restrict__ olat, int chunk, float* __restrict__ part) {
-  extern __shared__ float smem[];
+__global__ void __launch_bounds__(NACC > 8 ? 512 : 1024)
+latent_attention_kernel(const float* __restrict__ qfull, const T* __restrict__ pool, Paging pg, const Item* __restrict__ items, int H, int R, int dr, float scale,
+                        int window, const float* __restrict__ gate, int gate_ld, int gate_col0, const T* __restrict__ sink, T* __restrict__ olat, int chunk,
+                        float* __restrict__ part, int nbuf) {
+  extern __shared__ __align__(16) uint32_t lsm[];
+  constexpr int VPW = 4 / sizeof(T);                // values per word
   const Item it = items[blockIdx.x];
-  const int W = R + dr, WS = W | 1;                 // odd row stride: lane j reading row j is conflict-free
-  float* ktile = smem;                              // [32][WS]
-  float* qs = smem + 32 * WS;                       // [warps][W]
+  const int W = R + dr, WS = latent_row_words<T>(W), QS = (W + 3) & ~3;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int pair = blockIdx.y * nw + warp;         // (row, head) pair of this warp
   const bool active = pair < it.n_rows * H;
   const int qi = active ? pair / H : 0, h = active ? pair % H : 0;
   const int m = it.row0 + qi, pos = it.pos0 + qi;
-  float* q = qs + (size_t)warp * W;
-  if (active) {
-    const float* src = qfull + ((size_t)m * H + h) * W;
-    for (int d = lane; d < W; d += 32) q[d] = src[d];
-  }
+  float* q = reinterpret_cast<float*>(lsm + (size_t)nbuf * 32 * WS) + (size_t)warp * QS;
   int last = it.pos0 + it.n_rows - 1;
   int first = window > 0 ? max(0, it.pos0 - window + 1) : 0;
   if (gridDim.z > 1) {
     first += blockIdx.z * chunk;
     last = min(last, first + chunk - 1);
   }
+  // rows of a tile past `last` are neither loaded nor read
+  auto issue = [&](int j0, int b) {
+    for (int jr = warp; jr < 32 && j0 + jr <= last; jr += nw) {   // one warp per row
+      const T* src = pool + pg.row(it.slot, j0 + jr) * (size_t)W;
+      uint32_t* dst = lsm + (size_t)b * 32 * WS + jr * WS;
+      if (W % VPW == 0) {
+        for (int d = lane; d < W / VPW; d += 32) cp_async4(reinterpret_cast<float*>(dst + d), reinterpret_cast<const float*>(src + d * VPW));
+      } else {
+        for (int d = lane; d < W; d += 32) reinterpret_cast<T*>(dst)[d] = src[d];
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int ntile = last >= first ? (last - first) / 32 + 1 : 0;
+  if (ntile > 0) issue(first, 0);
+  if (active) {
+    const float* src = qfull + ((size_t)m * H + h) * W;
+    for (int d = lane; d < QS; d += 32) q[d] = d < W ? src[d] : 0.f;
+  }
   float acc[NACC];
 #pragma unroll
   for (int a = 0; a < NACC; ++a) acc[a] = 0.f;
   float mx = -INFINITY, den = 0.f;
-  for (int j0 = first; j0 <= last; j0 += 32) {
+  for (int t = 0; t < ntile; ++t) {
+    const int j0 = first + t * 32, b = nbuf > 1 ? t & 1 : 0;
+    if (nbuf > 1 && t + 1 < ntile) {
+      issue(j0 + 32, b ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
     __syncthreads();
-    // stage 32 cached rows (fp32), one warp per row — rows past `last` are zero-filled
-    for (int jr = warp; jr < 32; jr += nw) {
-      const int j = j0 + jr;
-      float* dst = ktile + jr * WS;
-      if (j <= last) {
-        const T* src = pool + pg.row(it.slot, j) * (size_t)W;
-        for (int d = lane; d < W; d += 32) dst[d] = ldf(src + d);
-      } else {
-        for (int d = lane; d < W; d += 32) dst[d] = 0.f;
+    if (active) {
+      const uint32_t* tile = lsm + (size_t)b * 32 * WS;
+      const int j = j0 + lane, n = min(32, last - j0 + 1);
+      const bool vis = j <= pos && j <= last && (window == 0 || pos - j < window);
+      const uint32_t* kr = tile + lane * WS;
+      float sp[4] = {0.f, 0.f, 0.f, 0.f};           // four independent partial sums
+      const int W4 = W / 4;
+#pragma unroll 4
+      for (int d = 0; d < W4; ++d) {
+        const float4 qv = *reinterpret_cast<const float4*>(q + 4 * d);
+        float kv[4];
+#pragma unroll
+        for (int x = 0; x < 4 / VPW; ++x) word_values<T>(kr[d * (4 / VPW) + x], kv + x * VPW);
+        sp[0] = fmaf(qv.x, kv[0], sp[0]);
+        sp[1] = fmaf(qv.y, kv[1], sp[1]);
+        sp[2] = fmaf(qv.z, kv[2], sp[2]);
+        sp[3] = fmaf(qv.w, kv[3], sp[3]);
+      }
+      for (int d = W4 * 4; d < W; ++d) sp[0] = fmaf(q[d], ldf(reinterpret_cast<const T*>(kr) + d), sp[0]);
+      const float s = vis ? ((sp[0] + sp[1]) + (sp[2] + sp[3])) * scale : -INFINITY;
+      const float tmax = warp_max(s);
+      if (tmax != -INFINITY) {                      // some key of the tile is visible (warp-uniform)
+        const float nmx = fmaxf(mx, tmax);
+        const float corr = expf(mx - nmx);          // mx == -inf: exp(-inf) = 0
+        const float p = vis ? expf(s - nmx) : 0.f;
+        den = den * corr + warp_sum(p);
+        mx = nmx;
+#pragma unroll
+        for (int a = 0; a < NACC; ++a) acc[a] *= corr;
+#pragma unroll 2
+        for (int jr = 0; jr < n; ++jr) {
+          const float pj = __shfl_sync(0xffffffffu, p, jr);
+          const uint32_t* c = tile + jr * WS;
+#pragma unroll
+          for (int a = 0; a < NACC / VPW; ++a) {    // word a * 32 + lane: latent columns VPW * (a * 32 + lane) ..
+            const int w = a * 32 + lane;
+            if (w * VPW < R) {
+              float v[VPW];
+              word_values<T>(c[w], v);
+#pragma unroll
+              for (int x = 0; x < VPW; ++x) acc[a * VPW + x] = fmaf(pj, v[x], acc[a * VPW + x]);
+            }
+          }
+        }
       }
     }
     __syncthreads();
-    if (!active) continue;
-    const int j = j0 + lane;
-    const bool vis = j <= pos && j <= last && (window == 0 || pos - j < window);
-    float s = 0.f;
-    const float* kr = ktile + lane * WS;
-    for (int d = 0; d < W; ++d) s = fmaf(q[d], kr[d], s);
-    s = vis ? s * scale : -INFINITY;
-    const float tmax = warp_max(s);
-    if (tmax == -INFINITY) continue;                // no visible key in this tile (warp-uniform)
-    const float nmx = fmaxf(mx, tmax);
-    const float corr = expf(mx - nmx);              // mx == -inf: exp(-inf) = 0
-    const float p = vis ? expf(s - nmx) : 0.f;
-    den = den * corr + warp_sum(p);
-    mx = nmx;
-#pragma unroll
-    for (int a = 0; a < NACC; ++a) acc[a] *= corr;
-    for (int jr = 0; jr < 32; ++jr) {
-      const float pj = __shfl_sync(0xffffffffu, p, jr);
-      if (pj == 0.f) continue;                      // warp-uniform
-      const float* c = ktile + jr * WS;
-#pragma unroll
-      for (int a = 0; a < NACC; ++a) {
-        const int d = a * 32 + lane;
-        if (d < R) acc[a] = fmaf(pj, c[d], acc[a]);
-      }
-    }
+    if (nbuf == 1 && t + 1 < ntile) issue(j0 + 32, 0);
   }
   if (!active) return;
   if (gridDim.z > 1) {
@@ -375,7 +441,7 @@ __global__ void latent_attention_kernel(const float* __restrict__ qfull, const T
     if (lane == 0) { dst[0] = mx; dst[1] = den; }
 #pragma unroll
     for (int a = 0; a < NACC; ++a) {
-      const int d = a * 32 + lane;
+      const int d = (a / VPW * 32 + lane) * VPW + a % VPW;
       if (d < R) dst[2 + d] = acc[a];
     }
     return;
@@ -386,12 +452,13 @@ __global__ void latent_attention_kernel(const float* __restrict__ qfull, const T
   T* out = olat + ((size_t)m * H + h) * R;
 #pragma unroll
   for (int a = 0; a < NACC; ++a) {
-    const int d = a * 32 + lane;
+    const int d = (a / VPW * 32 + lane) * VPW + a % VPW;
     if (d < R) stf(out + d, acc[a] * g);
   }
 }
 
-// merges the key runs of latent_attention_kernel: one warp per (row, head) pair of the listed items (grid.y covers the pairs);
+// merges the key runs of latent_attention_kernel: one warp per (row, head) pair of the listed items (grid.y covers the pairs) and 32-column
+// piece (grid.z);
 // lane z first turns run z's {max, sum} into its weight exp(max_z - max) (at most 32 runs), then the lanes split the R columns.  A
 // sink joins here, once, like a run that holds the weight exp(sink) and no values.
 template <typename T>
@@ -410,7 +477,7 @@ __global__ void latent_attention_combine_kernel(const float* __restrict__ part, 
   const float den = warp_sum(lane < splits ? src[(size_t)lane * (2 + R) + 1] * wz : 0.f) + (sink ? expf(sk - mx) : 0.f);
   float g = 1.0f / den;
   if (gate) g *= sigmoidf_(gate[(size_t)m * gate_ld + gate_col0 + h]);
-  for (int d0 = 0; d0 < R; d0 += 32) {
+  for (int d0 = blockIdx.z * 32; d0 < R; d0 += gridDim.z * 32) {
     const int d = d0 + lane;
     float a = 0.f;
 #pragma unroll 8
@@ -455,13 +522,6 @@ __global__ void delta_prepare_kernel(const float* __restrict__ proj, int ld, int
     au_out[o] = sigmoidf_(pr[col_a + h * dk + i] + ldf(a_bias + h * dk + i)) * u;
     wlog[o] = expf(-0.60653065971263342f * sigmoidf_(wlog[o] + ldf(w_bias + h * dk + i)));
   }
-}
-
-__device__ __forceinline__ void cp_async4(float* dst_smem, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst_smem)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async16(float* dst_smem, const float* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst_smem)), "l"(src) : "memory");
 }
 
 // A thread owns NC value columns x KPT key rows of the state (row i = e * P + part), so the token's vectors, read from shared
@@ -699,12 +759,11 @@ __global__ void __launch_bounds__(256)
 gemv_rows_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __restrict__ B, long sbn, long b_batch, TC* __restrict__ C, long ldc,
                  long c_batch, int M, int N, int K, int wsplit, const EpiArgs epi) {
   constexpr int RB = 4;
-  extern __shared__ float a_s[];                     // [M][K], then the slice sums [8 warps][RB][MR]
+  extern __shared__ __align__(16) float a_s[];       // [M][K], then the slice sums [8 warps][RB][MR]
   A += (size_t)blockIdx.z * a_batch;
   B += (size_t)blockIdx.z * b_batch;
   C += (size_t)blockIdx.z * c_batch;
-  for (int m = 0; m < M; ++m)
-    for (int k = threadIdx.x; k < K; k += blockDim.x) a_s[m * K + k] = ldf(A + (size_t)m * lda + k);
+  for (int m = 0; m < M; ++m) stage_f32(a_s + (size_t)m * K, A + (size_t)m * lda, K);
   float* red = a_s + (size_t)M * K;
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -741,16 +800,18 @@ gemv_rows_kernel(const TA* __restrict__ A, long lda, long a_batch, const TB* __r
         for (int u = 0; u < 2; ++u) {
           const int ku = min(k + u * 32 * VEC, K - VEC);     // past the slice the weights read as zero; the index stays inside a_s
 #pragma unroll
-          for (int v = 0; v < VEC; ++v) {
-            float av[MR];
+          for (int v = 0; v < VEC; v += 4) {
+            float av[MR][4];
 #pragma unroll
-            for (int m = 0; m < MR; ++m) av[m] = m < M ? a_s[m * K + ku + v] : 0.f;
+            for (int m = 0; m < MR; ++m) *reinterpret_cast<float4*>(av[m]) = m < M ? *reinterpret_cast<const float4*>(a_s + m * K + ku + v) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-            for (int r = 0; r < RB; ++r) {
-              const float w = ldf(reinterpret_cast<const TB*>(&raw[u][r]) + v);
+            for (int x = 0; x < 4; ++x)
 #pragma unroll
-              for (int m = 0; m < MR; ++m) acc[r][m] = fmaf(av[m], w, acc[r][m]);
-            }
+              for (int r = 0; r < RB; ++r) {
+                const float w = ldf(reinterpret_cast<const TB*>(&raw[u][r]) + v + x);
+#pragma unroll
+                for (int m = 0; m < MR; ++m) acc[r][m] = fmaf(av[m][x], w, acc[r][m]);
+              }
           }
         }
       }
