@@ -154,6 +154,18 @@ def test_unequal_requests_in_one_batch_equal_each_alone(dtype):
   n.close()
 
 
+def test_many_requests_in_one_step():
+  """more than a thousand rows (a count that is no multiple of four) in one step: the router then takes several rows per block"""
+  cfg = config([attention(heads=2, kv_heads=1, dim=8, vdim=8, mlp=moe(8, 2, (4, 2), 12))], width=48)
+  W = bo.random_weights(cfg, 14)
+  seqs = [rand_tokens(cfg["vocab"], 101, 200 + i) for i in range(13)]
+  n = make_engine(cfg, W, "float32", max_tokens=1400, max_requests=13, page_size=16)
+  lg, _ = n.step(list(range(13)), seqs, want=list(range(1313)))
+  for i in (0, 6, 12):
+    assert row_err(lg[101 * i:101 * (i + 1)], oracle_logits(cfg, W, seqs[i])[0]) < TOL["float32"]
+  n.close()
+
+
 def test_mixed_batch_of_portions_and_decoded_rows():
   cfg = config(MIXED)
   W = bo.random_weights(cfg, 6)

@@ -199,6 +199,20 @@ def test_unequal_requests_in_one_batch_equal_each_alone(dtype):
   n.close()
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_many_requests_in_one_step(dtype):
+  """more than a thousand rows (a count that is no multiple of four) in one step: the router then takes several rows per block"""
+  cfg = config([attn(heads=2, mlp=moe(8, 3, 16, (4, 2))), attn(mlp=moe(6, 2, 9, (3, 2)))], width=48)
+  W = ro.random_weights(cfg, 14)
+  seqs = [rand_tokens(cfg["vocab"], 101, 200 + i) for i in range(13)]
+  n = make_engine(cfg, W, dtype, max_tokens=1400, max_requests=13, page_size=16)
+  lg, _ = n.step(list(range(13)), seqs, want=list(range(1313)))
+  for i in (0, 6, 12):
+    ok = settled_rows(cfg, W, seqs[i], dtype)
+    assert ok.mean() > 0.5 and row_err(lg[101 * i:101 * (i + 1)][ok], oracle_logits(cfg, W, seqs[i])[0][ok]) < TOL[dtype]
+  n.close()
+
+
 def test_mixed_batch_of_portions_and_decoded_rows():
   cfg = config(MIXED)
   W = ro.random_weights(cfg, 6)

@@ -1331,12 +1331,16 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
       TRY((product<T, T, float, 0>(e, static_cast<T*>(e->act), s.shared_ff, 0, at<T>(e, L.down), s.shared_ff, 1, 0, e->y, D, 0, M, D, s.shared_ff, 1)));
     }
     {
-      auto kern = moe_router_kernel<T>;
-      const size_t rsm = ((size_t)((D + 3) & ~3) + (s.router_kind == XOTB200_LM_ROUTER_SIGMOID_GROUPS ? 2 * E + std::max(1, s.groups) : E)) * 4;
+      // several rows per block when there are enough for all SMs and they fit in shared memory
+      constexpr int RPB = 4;
+      const size_t row_sm = ((size_t)((D + 3) & ~3) + moe_router_scores(s.router_kind, E, s.groups)) * 4;
+      const bool multi = M >= RPB * e->sm_count && RPB * row_sm <= 100 * 1024;
+      auto kern = multi ? moe_router_kernel<T, RPB> : moe_router_kernel<T, 1>;
+      const size_t rsm = (multi ? RPB : 1) * row_sm;
       TRY(opt_in_smem(kern, rsm));
-      kern<<<M, std::min(1024, std::max(64, (M <= 16 ? E : cdiv(E, 2)) * 32)), rsm, e->stream>>>(h, D, at<T>(e, L.router), s.router_bias ? at<T>(e, L.router_b) : nullptr,
-                                                                                 s.router_kind, E, s.groups, s.groups_keep, top, s.router_correction ? at<T>(e, L.correction) : nullptr,
-                                                                                 s.group_best, s.router_scale, e->moe_ids, e->moe_wts, M);
+      kern<<<multi ? cdiv(M, RPB) : M, std::min(1024, std::max(32 * RPB, (M <= 16 ? E : cdiv(E, 2)) * 32)), rsm, e->stream>>>(
+          h, D, at<T>(e, L.router), s.router_bias ? at<T>(e, L.router_b) : nullptr, s.router_kind, E, s.groups, s.groups_keep, top,
+          s.router_correction ? at<T>(e, L.correction) : nullptr, s.group_best, s.router_scale, e->moe_ids, e->moe_wts, M);
     }
     CK(cudaGetLastError());
     e->launches++;

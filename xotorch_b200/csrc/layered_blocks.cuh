@@ -283,21 +283,8 @@ __device__ __forceinline__ void dot16(float& acc, const uint4& raw, const float*
   }
 }
 
-// dot product of a weight row (T, global) with a row held in shared memory (fp32), 16 bytes per lane per load when `vec` (which also says
-// that the row in shared memory is on a 16-byte boundary)
-template <typename T>
-__device__ __forceinline__ float row_dot(const T* __restrict__ w, const float* __restrict__ xs, int n, int lane, bool vec) {
-  constexpr int VEC = 16 / sizeof(T);
-  float acc = 0.f;
-  if (vec) {
-#pragma unroll 4
-    for (int k = lane * VEC; k < n; k += 32 * VEC) dot16<T>(acc, *reinterpret_cast<const uint4*>(w + k), xs + k);
-  } else {
-    for (int k = lane; k < n; k += 32) acc = fmaf(ldf(w + k), xs[k], acc);
-  }
-  return warp_sum(acc);
-}
-
+// Dot products of a weight row (T, global) with one or two rows of x held in shared memory (fp32), 16 bytes per lane per load when `vec` (which
+// also says that the rows in shared memory are on 16-byte boundaries).
 // two rows at once (w0 . x0 and w1 . x1): twice the loads in flight
 template <typename T>
 __device__ __forceinline__ void row_dot2(const T* __restrict__ w0, const T* __restrict__ w1, const float* __restrict__ x0, const float* __restrict__ x1,
@@ -407,27 +394,61 @@ __device__ __forceinline__ int warp_argmax(const float* v, int n, int lane) {
 //   kind 2: scores s = sigmoid(z), CHOICE scores c = s + correction (may be negative); a group's score is the sum of its `group_best`
 //           largest c, only experts of the `keep` best groups can be chosen; the `top` largest c of those are the token's experts,
 //           weighted by their s over the sum of the chosen s, times wscale.  The whole warp selects.
-// Ties go to the lower index.  One block per row (its warps share the experts' logits, warp 0 selects); dynamic shared memory:
-// D + E floats (kind 2: D + 2 E + groups).
+// Ties go to the lower index.  One block per RPB rows (with many rows the router's matrix is read once for all of them); its warps share
+// the experts' logits, then warp r selects for row r.  Dynamic shared memory: RPB x (D + moe_router_scores) floats.
 // ---------------------------------------------------------------------------------------------------------------------------
-template <typename T>
-__global__ void moe_router_kernel(const T* __restrict__ h, int D, const T* __restrict__ w_router, const T* __restrict__ bias, int kind, int E,
+__host__ __device__ __forceinline__ int moe_router_scores(int kind, int E, int groups) { return kind == 2 ? 2 * E + (groups > 1 ? groups : 1) : E; }
+
+template <typename T, int RPB>
+__global__ void __launch_bounds__(1024) moe_router_kernel(const T* __restrict__ h, int D, const T* __restrict__ w_router, const T* __restrict__ bias, int kind, int E,
                                   int groups, int keep, int top, const T* __restrict__ correction, int group_best, float wscale, int* __restrict__ ids,
                                   float* __restrict__ wts, int M) {
-  extern __shared__ __align__(16) float rsm[];                 // [D] the row (fp32), then [E] scores
+  extern __shared__ __align__(16) float rsm[];                 // [RPB][D] the rows (fp32), then [RPB] scores
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const int m = blockIdx.x;
-  float* hs = rsm;
-  float* s = rsm + ((D + 3) & ~3);
-  stage_f32(hs, h + (size_t)m * D, D);
+  const int m0 = blockIdx.x * RPB, nr = min(RPB, M - m0), Dp = (D + 3) & ~3, ns = moe_router_scores(kind, E, groups);
+  float* scores = rsm + RPB * Dp;
+#pragma unroll
+  for (int r = 0; r < RPB; ++r)
+    if (r < nr) stage_f32(rsm + r * Dp, h + (size_t)(m0 + r) * D, D);
   __syncthreads();
-  const bool vec = D % (16 / sizeof(T)) == 0 && (reinterpret_cast<uintptr_t>(w_router) & 15) == 0;
+  constexpr int VEC = 16 / sizeof(T), NB = RPB > 1 ? 2 : 4;     // NB weight pieces in flight per lane
+  const bool vec = D % VEC == 0 && (reinterpret_cast<uintptr_t>(w_router) & 15) == 0;
   for (int e = warp; e < E; e += nw) {                         // the warps share the experts; logits in fp32
-    const float z = row_dot(w_router + (size_t)e * D, hs, D, lane, vec);
-    if (lane == 0) s[e] = z + (bias ? ldf(bias + e) : 0.f);
+    const T* w = w_router + (size_t)e * D;
+    float z[RPB];
+#pragma unroll
+    for (int r = 0; r < RPB; ++r) z[r] = 0.f;
+    if (vec) {
+      for (int k = lane * VEC; k < D; k += 32 * VEC * NB) {
+        uint4 raw[NB];
+#pragma unroll
+        for (int b = 0; b < NB; ++b) raw[b] = k + b * 32 * VEC < D ? *reinterpret_cast<const uint4*>(w + k + b * 32 * VEC) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+          const int kb = k + b * 32 * VEC < D ? k + b * 32 * VEC : k;   // past the end the weights read as zero; the index stays inside the row
+#pragma unroll
+          for (int r = 0; r < RPB; ++r)
+            if (r < nr) dot16<T>(z[r], raw[b], rsm + r * Dp + kb);
+        }
+      }
+    } else {
+      for (int k = lane; k < D; k += 32) {
+        const float wv = ldf(w + k);
+#pragma unroll
+        for (int r = 0; r < RPB; ++r)
+          if (r < nr) z[r] = fmaf(wv, rsm[r * Dp + k], z[r]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < RPB; ++r) {
+      z[r] = warp_sum(z[r]);
+      if (lane == 0) scores[r * ns + e] = z[r] + (bias ? ldf(bias + e) : 0.f);
+    }
   }
   __syncthreads();
-  if (warp != 0) return;
+  if (warp >= nr) return;
+  const size_t m = m0 + warp;
+  float* s = scores + warp * ns;
   if (kind == 1) {
     if (lane == 0) {
       float den = 0.f, first = 0.f;
