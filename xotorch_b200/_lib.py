@@ -183,7 +183,7 @@ def load_lm(path: os.PathLike | None = None, build: bool = True) -> C.CDLL:
   p = Path(path) if path else Path(os.environ.get("XOTB200_LM_LIB", LM_LIB_PATH))
   if build and path is None and "XOTB200_LM_LIB" not in os.environ:
     src = Path(__file__).resolve().parent / "csrc"
-    deps = [src / n for n in ("layered.cu", "layered_kernels.cuh", "layered_blocks.cuh", "layered_gqa.cuh", "layered_tc.cuh", "prefill_tc.cuh", "kernels.cuh", "st_header.h")]
+    deps = [src / n for n in ("layered.cu", "layered_kernels.cuh", "layered_blocks.cuh", "layered_gqa.cuh", "layered_recurrent.cuh", "layered_tc.cuh", "prefill_tc.cuh", "kernels.cuh", "st_header.h")]
     deps.append(src.parent.parent / "include" / "xotb200_lm.h")
     stale = p.exists() and any(d.exists() and d.stat().st_mtime > p.stat().st_mtime for d in deps)
     if not p.exists() or stale:
