@@ -12,7 +12,8 @@
  *   XOTB200_LM_MIX_ATTENTION    grouped-query attention over a paged cache of (normed) keys and values; options: projection
  *                               biases, query/key norm (per head or over the whole projection), soft cap, logarithmic distance
  *                               penalty, learned bias per distance bucket, query temperature, softmax sink, sliding window,
- *                               block-local mask, output gate per head or per entry, keys/values borrowed from an earlier layer;
+ *                               block-local mask, output gate per head or per entry, keys/values borrowed from an earlier layer,
+ *                               short convolutions on the projections, values mixed with those of an earlier layer;
  *   XOTB200_LM_MIX_GATED_DELTA  delta rule with one decay per head behind short causal convolutions;
  *                               state = fp32 matrix per head + the convolutions' last inputs;
  *   XOTB200_LM_MIX_MATRIX_LSTM  matrix memory with exponential input gate, sigmoid forget gate and a running maximum that keeps both
@@ -25,7 +26,8 @@
  * A layer wraps its sublayers in grouped RMS norms before and after them, or reads the stream itself and closes with a layer norm
  * or an RMS norm, or — pre-norm with one-number weights — reads `streams` copies of the residual stream through hyper-connections
  * and passes every sublayer input through a short causal convolution that is added to it, or — pre-norm with a Dynamic Tanh —
- * norms every entry of the stream by itself (xotb200_lm_cfg.block); its feed-forward is dense (relu^2, xIELU, gelu, gated gelu) or a
+ * norms every entry of the stream by itself, or — parallel — feeds one RMS-normed input to its mixer and its feed-forward and adds both
+ * results to the stream (xotb200_lm_cfg.block); its feed-forward is dense (relu^2, xIELU, gelu, gated gelu, clamped gated) or a
  * mixture of experts (gated silu, clamped gated or relu^2 experts, three routing rules, an optional shared expert:
  * xotb200_lm_layer.ff_kind and the fields after it).  A layer may use another layer's weights (weights_of) with a cache / state of its own.
  * Every size and constant of a layer is a field of xotb200_lm_layer, so a model family is a table of layers, not code.
@@ -70,6 +72,8 @@ extern "C" {
                                   p, q = the two entries of l<i>.mlp.act                                                         */
 #define XOTB200_LM_FF_GELU 3   /* W_down gelu(W_up h), the exact gelu z (1 + erf(z / sqrt 2)) / 2                               */
 #define XOTB200_LM_FF_GELU_GATED 4 /* W_down (gelu_tanh(W_gate h) * W_up h), the tanh form of gelu                                */
+#define XOTB200_LM_FF_CLAMPED_GLU 5 /* W_down (g sigmoid(slope g) (u + 1)), g = min(W_gate h, limit), u = W_up h clamped to [-limit, limit]
+                                       (expert_limit, expert_slope)                                                                   */
 #define XOTB200_LM_FF_MOE 2    /* mixture of experts; expert form, routing rule and shared expert: expert_act, router_kind, shared_ff */
 
 #define XOTB200_LM_EXPERT_SILU_GATED 0 /* expert = W_down (silu(W_gate h) * W_up h)                                              */
@@ -94,10 +98,20 @@ extern "C" {
 #define XOTB200_LM_BLOCK_PRE_DYT 4     /* x += ls * sublayer(tanh(alpha x) * w + b): pre-norm by a Dynamic Tanh (no statistic of the row), the
                                          sublayer's result scaled entry by entry when layer_scale; the final norm of the same kind      */
 
+#define XOTB200_LM_BLOCK_PARALLEL_RMS 5  /* h = rms(x) * w, x += mixer(h) + ff(h): one plain RMS norm per layer (norm1), both sublayers read it;
+                                           the final norm of the same kind                                                        */
+
 #define XOTB200_LM_QKNORM_NONE 0
 #define XOTB200_LM_QKNORM_HEAD 1      /* RMS norm of every query / key head, one weight of size dim shared by the heads                 */
 #define XOTB200_LM_QKNORM_HEAD_PLAIN 3 /* every query / key head divided by its root mean square, no weight                            */
+#define XOTB200_LM_QKNORM_HEAD_ROTATED 4 /* the same after the rotation: every ROTATED query / key head divided by its root mean square      */
 #define XOTB200_LM_QKNORM_ROW 2       /* ONE RMS norm over the whole query (key) projection, weights of size heads * dim (kv_heads * dim) */
+
+#define XOTB200_LM_SINK_LEARNED 1 /* `sink`: the softmax denominator also holds exp(sink[a]), one learned number per query head          */
+#define XOTB200_LM_SINK_ONE 2     /* `sink`: the softmax denominator also holds 1 (a sink whose score is 0)                              */
+
+#define XOTB200_LM_ROT_SCALE_WAVELENGTH 0 /* rot_scale_kind: see rot_scale_factor                                                 */
+#define XOTB200_LM_ROT_SCALE_YARN 1       /* rot_scale_kind: see rot_scale_kind                                                   */
 
 #define XOTB200_LM_ROT_INTERLEAVED 0 /* pairs (2i, 2i+1)        */
 #define XOTB200_LM_ROT_HALF 1        /* pairs (i, i + dims / 2) */
@@ -134,7 +148,9 @@ typedef struct xotb200_lm_layer {
   int32_t qk_norm;    /* attention: XOTB200_LM_QKNORM_* (weights q.norm / k.norm)                              */
   int32_t proj_bias;  /* attention: 1 = q, k, v projections have biases (q.b, k.b, v.b)                       */
   int32_t dist_bias;  /* attention: 1 = logarithmic distance penalty with per-head r1, r2                     */
-  int32_t conv_taps;  /* gated delta rule: taps of the short convolutions                                     */
+  int32_t conv_taps;  /* gated delta rule: taps of the short convolutions; attention: > 0 = every channel of the q, k and v projections (bias
+                         included) passes a causal filter of this many taps (q.conv, k.conv, v.conv) before norm and rotation; the filters'
+                         last inputs are part of the request's state                                          */
   int32_t ff_kind;    /* XOTB200_LM_FF_*  (`ff` = inner size of the dense forms)                              */
   int32_t experts;    /* FF_MOE: number of experts, each of inner size expert_ff                              */
   int32_t expert_ff;
@@ -144,7 +160,7 @@ typedef struct xotb200_lm_layer {
   float softcap;
   /* -- further options of MIX_ATTENTION -------------------------------------------------------------------------------- */
   int32_t out_bias;     /* 1 = the output projection has a bias (o.b)                                            */
-  int32_t sink;         /* 1 = one learned logit per query head (sink) joins the softmax denominator            */
+  int32_t sink;         /* 0 none, else XOTB200_LM_SINK_*: a term without key or value joins the softmax denominator */
   int32_t rel_buckets;  /* B > 0: learned bias rel[B, heads] per distance bucket.  With h = B / 2 (integer): distances n < h have a
                            bucket each (n); the other B - h buckets divide [h, rel_max] in equal steps of ln(n):
                            bucket = min(B - 1, h + floor((B - h) * ln(n / h) / ln(rel_max / h)))                 */
@@ -199,6 +215,14 @@ typedef struct xotb200_lm_layer {
   int32_t router_correction; /* ROUTER_SIGMOID_GROUPS: 1 = choice scores have a correction per expert (mlp.correction)   */
   int32_t group_best;     /* ROUTER_SIGMOID_GROUPS: how many of a group's largest choice scores make its score (1 or 2) */
   float router_scale;     /* ROUTER_SIGMOID_GROUPS: factor of the normalised weights                                */
+  /* -- further options of MIX_ATTENTION -------------------------------------------------------------------------------------------
+   * rot_scale_kind = ROT_SCALE_YARN (with rot_scale_factor > 0; rot_scale_low / rot_scale_high = turns over the original length): let
+   * at(t) = dims ln(original / (2 pi t)) / (2 ln base), a = max(floor(at(high)), 0), b = min(ceil(at(low)), dims - 1); frequency i is
+   * blended from f_i (i <= a) to f_i / factor (i >= b) linearly in i, and cosines and sines are multiplied by 0.1 ln(factor) + 1.
+   * v_mix = 1: value mixing.  The first layer of the model with v_mix hands its values to the later ones: there
+   * v <- (1 - c) v + c v_first with c = l<i>.mix.vmix (one number), before v is cached; equal kv_heads and vdim in all of them. */
+  int32_t rot_scale_kind;
+  int32_t v_mix;
 } xotb200_lm_layer;
 
 typedef struct xotb200_lm_cfg {
@@ -227,6 +251,12 @@ typedef struct xotb200_lm_cfg {
   float residual_mult;   /* 0 = 1                                                                                                   */
   int32_t layer_scale;   /* BLOCK_PRE_DYT: 1 = a sublayer's result is multiplied entry by entry by l<i>.ls1 / ls2 before the sum          */
   int32_t tied_head;     /* 1 = the logits use the embedding table (no tensor `head`)                                               */
+  /* -- BLOCK_PARALLEL_RMS: the embedding ------------------------------------------------------------------------------------------ */
+  float embed_scale;     /* the embedding row is multiplied by this (0 = 1); a tied head uses the table without it                        */
+  int32_t bigram_buckets;/* B > 0: row (previous token * bigram_mul_prev + token * bigram_mul_cur) mod B of the table `bigram` [B + 1, width] is
+                            added, row B for the first token of a request (the previous token is part of the request's state)             */
+  int64_t bigram_mul_prev;
+  int64_t bigram_mul_cur;
 } xotb200_lm_cfg;
 
 typedef struct xotb200_lm xotb200_lm;
@@ -250,6 +280,8 @@ int xotb200_lm_destroy(xotb200_lm* e);
  * .mix; MIX_ATTENTION with QKNORM_HEAD_PLAIN has no norm weights; MIX_MATRIX_LSTM <t> in {q, k, v, g, i, i.b, f, f.b, norm, o};
  * BLOCK_PRE_DYT models: norm weights <norm>, <norm>.alpha (one number), <norm>.b for l<i>.norm1 / norm2 and final.norm; l<i>.ls1 / ls2;
  * MIX_LATENT_ATTN with a sink: sink [heads]; FF_GELU_GATED: mlp.gate / up / down; ROUTER_SIGMOID_GROUPS: mlp.correction [experts].
+ * BLOCK_PARALLEL_RMS models: bigram, l<i>.norm1, final.norm; MIX_ATTENTION with conv_taps: q.conv / k.conv / v.conv [channels, taps], with v_mix:
+ * vmix (one number); FF_CLAMPED_GLU: mlp.gate / up / down.
  * MIX_MAMBA2 <t> in {in, conv, conv.b, dt_bias, A_log, D, norm, o}; a layer with two mixers names them l<i>.mix.left.<t> / .right.<t>.
  * xotb200_lm_load_dir reads every *.safetensors of the directory (BF16 tensors) and is STRICT: a tensor of this shard that is
  * missing, has another shape or dtype, or an unknown tensor of an owned layer, is an error. */
@@ -268,14 +300,19 @@ int xotb200_lm_clear_request(xotb200_lm* e, int slot);
 int xotb200_lm_request_len(xotb200_lm* e, int slot, int* len);
 
 /* The step.  n_seq requests; request i is slot slots[i] and brings counts[i] >= 1 rows, which continue it at its current length.
- * First shard: tokens[sum counts] (int32 ids); other shards: hidden_f32[sum counts, width] (the fp32 residual stream).
+ * First shard: tokens[sum counts] (int32 ids); other shards: hidden_f32[sum counts, width] (the fp32 residual stream, followed row by
+ * row by the first mixing layer's values when that layer is in an earlier shard: see xotb200_lm_hidden_width).
  * want_rows[n_want]: indices into the packed rows whose output is asked for.
  *   last shard : logits_f32[n_want, vocab] and/or argmax_i32[n_want] (lowest-index argmax) — either may be NULL;
- *   other shards: hidden_out_f32[sum counts, width] (want_rows ignored).
+ *   other shards: hidden_out_f32[sum counts, width] (want_rows ignored; with the values that a later shard's layers mix in).
  * A slot may appear once per step.  Fails without touching any state when the pool has too few free pages. */
 int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_t* counts, const int32_t* tokens,
                     const float* hidden_f32, const int32_t* want_rows, int n_want, float* logits_f32, int32_t* argmax_i32,
                     float* hidden_out_f32);
+
+/* floats per row of hidden_f32 (*in; 0 on the first shard) and hidden_out_f32 (*out; 0 on the last): the width, plus kv_heads * vdim where the
+ * first mixing layer's values (v_mix) have to cross the shard border */
+int xotb200_lm_hidden_width(xotb200_lm* e, int* in, int* out);
 
 /* Debug / tests: the fp32 residual stream after every layer of the most recent step is kept when enabled (trace = 1) and copied
  * out as [local layers, rows, width]. */

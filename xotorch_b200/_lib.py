@@ -101,11 +101,13 @@ def load(path: os.PathLike | None = None) -> C.CDLL:
 LM_LIB_PATH = Path(__file__).resolve().parent / "lib" / "libxotb200_lm.so"
 LM_DTYPE_BF16, LM_DTYPE_F32 = 0, 2
 LM_MIX_LATENT_ATTN, LM_MIX_DELTA_RULE, LM_MIX_ATTENTION, LM_MIX_GATED_DELTA, LM_MIX_MATRIX_LSTM, LM_MIX_MAMBA2 = 0, 1, 2, 3, 4, 5
-LM_FF_RELU2, LM_FF_XIELU, LM_FF_MOE, LM_FF_GELU, LM_FF_GELU_GATED = 0, 1, 2, 3, 4
+LM_FF_RELU2, LM_FF_XIELU, LM_FF_MOE, LM_FF_GELU, LM_FF_GELU_GATED, LM_FF_CLAMPED_GLU = 0, 1, 2, 3, 4, 5
 LM_EXPERT_SILU_GATED, LM_EXPERT_RELU2, LM_EXPERT_CLAMPED_GLU = 0, 1, 2
 LM_ROUTER_SOFTMAX_ALL, LM_ROUTER_TOPK_SOFTMAX, LM_ROUTER_SIGMOID_GROUPS = 0, 1, 2
-LM_BLOCK_GROUP_RMS, LM_BLOCK_POST_LN, LM_BLOCK_POST_RMS, LM_BLOCK_PRE_SCALAR, LM_BLOCK_PRE_DYT = 0, 1, 2, 3, 4
-LM_QKNORM_NONE, LM_QKNORM_HEAD, LM_QKNORM_ROW, LM_QKNORM_HEAD_PLAIN = 0, 1, 2, 3
+LM_BLOCK_GROUP_RMS, LM_BLOCK_POST_LN, LM_BLOCK_POST_RMS, LM_BLOCK_PRE_SCALAR, LM_BLOCK_PRE_DYT, LM_BLOCK_PARALLEL_RMS = 0, 1, 2, 3, 4, 5
+LM_QKNORM_NONE, LM_QKNORM_HEAD, LM_QKNORM_ROW, LM_QKNORM_HEAD_PLAIN, LM_QKNORM_HEAD_ROTATED = 0, 1, 2, 3, 4
+LM_SINK_LEARNED, LM_SINK_ONE = 1, 2
+LM_ROT_SCALE_WAVELENGTH, LM_ROT_SCALE_YARN = 0, 1
 LM_ROT_INTERLEAVED, LM_ROT_HALF = 0, 1
 
 
@@ -127,7 +129,7 @@ class LmLayer(C.Structure):
     ("par_vdim", C.c_int32), ("par_conv_taps", C.c_int32), ("par_out_norm_groups", C.c_int32), ("par_gate_cap", C.c_float),
     ("mix_scale", C.c_float), ("par_scale", C.c_float),
     ("weights_of", C.c_int32), ("expert_limit", C.c_float), ("expert_slope", C.c_float), ("router_correction", C.c_int32),
-    ("group_best", C.c_int32), ("router_scale", C.c_float),
+    ("group_best", C.c_int32), ("router_scale", C.c_float), ("rot_scale_kind", C.c_int32), ("v_mix", C.c_int32),
   ]
 
 
@@ -137,7 +139,8 @@ class LmCfg(C.Structure):
     ("norm_groups", C.c_int32), ("dtype", C.c_int32), ("norm_eps", C.c_float), ("block", C.c_int32), ("max_positions", C.c_int32),
     ("pos_sinusoid", C.c_int32), ("sinusoid_base", C.c_float), ("embed_norm", C.c_int32), ("logit_scale", C.c_float),
     ("logit_softcap", C.c_float), ("streams", C.c_int32), ("canon_taps", C.c_int32), ("residual_mult", C.c_float),
-    ("layer_scale", C.c_int32), ("tied_head", C.c_int32),
+    ("layer_scale", C.c_int32), ("tied_head", C.c_int32), ("embed_scale", C.c_float), ("bigram_buckets", C.c_int32),
+    ("bigram_mul_prev", C.c_int64), ("bigram_mul_cur", C.c_int64),
   ]
 
 
@@ -156,6 +159,7 @@ _LM_SIGS = {
   "xotb200_lm_request_len": (C.c_int, [C.c_void_p, C.c_int, C.POINTER(C.c_int)]),
   "xotb200_lm_step": (C.c_int, [C.c_void_p, C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_void_p,
                                 C.c_void_p, C.c_void_p]),
+  "xotb200_lm_hidden_width": (C.c_int, [C.c_void_p, C.POINTER(C.c_int), C.POINTER(C.c_int)]),
   "xotb200_lm_set_trace": (C.c_int, [C.c_void_p, C.c_int]),
   "xotb200_lm_read_trace": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int64]),
   "xotb200_lm_set_gemm_mode": (C.c_int, [C.c_void_p, C.c_int]),

@@ -92,6 +92,9 @@ struct LmLayer {
   // grouped-query attention: columns of q / k / v (gate: c_g), bias vector over the projection's columns, norm weights, penalties
   int c_kk = 0, c_vv = 0;
   size_t b_in = 0, q_norm = 0, k_norm = 0, r1 = 0, r2 = 0, o_b = 0, sink = 0, rel = 0;
+  size_t vmix = 0;                                     // the number that mixes the values with the first mixing layer's
+  int vmix_mode = 0;                                   // 0 no mixing, 1 this layer hands its values on, 2 it mixes them in
+  float rot_mul = 1.f;                                 // factor of the rotation's cosines and sines
   int rel_n = 0;                                       // distances tabulated for the learned bias: every distance >= rel_n - 1 is in the last bucket
   int* rel_bucket = nullptr;                           // [rel_n] bucket of every tabulated distance (device; made on the host in double)
   float* rel_tab = nullptr;                            // [heads][rel_n] the bias per head and distance (device; remade when weights change)
@@ -165,6 +168,11 @@ struct xotb200_lm {
   int max_heads_rec = 0;
   bool pre_scalar = false;
   bool pre_dyt = false;
+  bool parallel = false;
+  size_t bigram = 0;                                   // hashed (previous token, token) table
+  std::vector<int> slot_last;                          // per slot: its newest token (the previous token of its next row)
+  float* vfirst = nullptr;                             // values of the first mixing layer, [rows, vfirst_n]
+  int vfirst_n = 0, carry_in = 0, carry_out = 0;       // its size; how many of its floats per row come from / go to the neighbouring shards
   size_t final_norm_b = 0, final_norm_a = 0, pos_table = 0;
   const EpiArgs* close = nullptr;                      // set by a block form whose sublayers close themselves in their last kernel; NULL: they write y
   bool closed = false;                                 // the sublayer that ran has done so
@@ -225,6 +233,22 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
   const int S = e->cfg.streams, CT = e->cfg.canon_taps;
   e->pre_scalar = pre_scalar;
   e->pre_dyt = pre_dyt;
+  const bool parallel = e->cfg.block == XOTB200_LM_BLOCK_PARALLEL_RMS;
+  e->parallel = parallel;
+  // value mixing: the model's first layer with v_mix hands its values to the later ones, across shard borders too
+  int v_first_layer = -1;
+  for (int li = 0; li < e->cfg.n_layers; ++li) {
+    if (!all[li].v_mix) continue;
+    REQUIRE(all[li].mixer == XOTB200_LM_MIX_ATTENTION && all[li].kv_from < 0, "layer %d: only attention with values of its own mixes values", li);
+    if (v_first_layer < 0) v_first_layer = li;
+    REQUIRE(all[li].kv_heads == all[v_first_layer].kv_heads && all[li].vdim == all[v_first_layer].vdim, "layer %d mixes in the values of layer %d, which has other sizes", li,
+            v_first_layer);
+    e->vfirst_n = all[li].kv_heads * all[li].vdim;
+    if (li > v_first_layer) {
+      if (v_first_layer < e->cfg.start_layer && li >= e->cfg.start_layer) e->carry_in = e->vfirst_n;
+      if (v_first_layer <= e->cfg.end_layer && li > e->cfg.end_layer) e->carry_out = e->vfirst_n;
+    }
+  }
   // what a sublayer of the pre-scalar block owns besides its norm: input convolution and hyper-connection coefficients
   auto sublayer_extras = [&](LmLayer& L, const std::string& p, int q) {
     const std::string n = std::to_string(q + 1);
@@ -251,6 +275,7 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
   if (e->first) {
     e->embed = take((size_t)V * D); dest("embed", e->embed, V, D, 0);
     if (e->cfg.embed_norm) { e->embed_norm = take(NW); dest("embed.norm", e->embed_norm, 1, NW, 0); }
+    if (e->cfg.bigram_buckets > 0) { e->bigram = take((size_t)(e->cfg.bigram_buckets + 1) * D); dest("bigram", e->bigram, e->cfg.bigram_buckets + 1, D, 0); }
     if (e->cfg.max_positions > 0) { e->pos_table = take((size_t)e->cfg.max_positions * D); dest("pos", e->pos_table, e->cfg.max_positions, D, 0); }
   }
   for (int li = e->cfg.start_layer; li <= e->cfg.end_layer; ++li) {
@@ -278,6 +303,7 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
       C.state_begin += shift;
       e->state_floats += C.state_size;
       C.s = s;
+      if (s.v_mix) C.vmix_mode = li == v_first_layer ? 1 : 2;
       if (s.mixer == XOTB200_LM_MIX_ATTENTION && s.kv_from < 0) C.kv_src = li - e->cfg.start_layer;
       e->layers.push_back(C);
       continue;
@@ -287,7 +313,7 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
     const std::string p = "l" + std::to_string(own_li) + ".";
     REQUIRE(s.heads >= 1 && s.dim >= 1, "layer %d: heads and dim must be positive", li);
     L.norm1 = take(NW); dest(p + "norm1", L.norm1, 1, NW, 0);
-    if (!post_rms && !pre_scalar) { L.norm1b = take(D); dest(p + "norm1" + nb, L.norm1b, 1, D, 0); }
+    if (!post_rms && !pre_scalar && !parallel) { L.norm1b = take(D); dest(p + "norm1" + nb, L.norm1b, 1, D, 0); }
     if (pre_scalar) sublayer_extras(L, p, 0);
     if (pre_dyt) dyt_extras(p, "1", L.norm1a, L.ls1);
     // one mixer: its projection columns start at column cb of the layer's projection output; `shared`: the projection matrix of
@@ -362,11 +388,17 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
       REQUIRE(dv >= 1 && dv <= 512 && dk <= 1024, "layer %d: attention sizes dim %d (<= 1024) / vdim %d (1..512)", li, dk, dv);
       REQUIRE(s.window >= 0 && s.chunk >= 0 && s.softcap >= 0.f, "layer %d: negative window, chunk or softcap", li);
       REQUIRE(s.out_gate >= 0 && s.out_gate <= 2, "layer %d: unknown output gate %d", li, s.out_gate);
-      REQUIRE(s.qk_norm >= XOTB200_LM_QKNORM_NONE && s.qk_norm <= XOTB200_LM_QKNORM_HEAD_PLAIN, "layer %d: unknown query/key norm %d", li, s.qk_norm);
+      REQUIRE(s.qk_norm >= XOTB200_LM_QKNORM_NONE && s.qk_norm <= XOTB200_LM_QKNORM_HEAD_ROTATED, "layer %d: unknown query/key norm %d", li, s.qk_norm);
       REQUIRE(s.rot_dims >= 0 && s.rot_dims <= dk && s.rot_dims % 2 == 0, "layer %d: %d rotated entries of a head of %d", li, s.rot_dims, dk);
       REQUIRE(s.rot_dims == 0 || (s.rot_base > 0.f && (s.rot_layout == XOTB200_LM_ROT_INTERLEAVED || s.rot_layout == XOTB200_LM_ROT_HALF)),
               "layer %d: rotation needs a positive base and a known layout", li);
       REQUIRE(s.rot_dims == 0 || s.qk_norm != XOTB200_LM_QKNORM_ROW, "layer %d: rotation is implemented with per-head query/key norms (or none)", li);
+      REQUIRE(s.rot_scale_kind == XOTB200_LM_ROT_SCALE_WAVELENGTH || s.rot_scale_kind == XOTB200_LM_ROT_SCALE_YARN, "layer %d: unknown frequency scaling %d", li, s.rot_scale_kind);
+      REQUIRE(s.rot_scale_kind != XOTB200_LM_ROT_SCALE_YARN || s.rot_dims == 0 || (s.rot_base != 1.f && s.rot_scale_factor > 0.f), "layer %d: YaRN scaling needs a base other than 1 and a factor", li);
+      REQUIRE(s.sink >= 0 && s.sink <= XOTB200_LM_SINK_ONE, "layer %d: unknown sink %d", li, s.sink);
+      REQUIRE(s.conv_taps >= 0 && s.conv_taps <= 64, "layer %d: %d convolution taps (0..64)", li, s.conv_taps);
+      REQUIRE((s.conv_taps == 0 && s.qk_norm != XOTB200_LM_QKNORM_HEAD_ROTATED && s.rot_scale_kind == 0) || (own && s.qk_norm != XOTB200_LM_QKNORM_ROW),
+              "layer %d: convolutions, a norm after the rotation and YaRN scaling go with keys/values of the layer's own and per-head norms", li);
       REQUIRE(s.rot_scale_factor == 0.f || (s.rot_scale_factor > 0.f && s.rot_scale_high > s.rot_scale_low && s.rot_scale_low > 0.f && s.rot_scale_original > 0.f),
               "layer %d: frequency scaling needs factor > 0, 0 < low < high and the original length", li);
       REQUIRE(s.keep_first >= 0 && s.pool >= 0 && !(s.keep_first > 0 && s.pool > 0), "layer %d: kept first tokens and pooled blocks exclude each other", li);
@@ -402,14 +434,28 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
         dest(mp + "q.b", L.b_in + L.c_q, 1, H * dk, 0);
         if (own) { dest(mp + "k.b", L.b_in + L.c_kk, 1, G * dk, 0); dest(mp + "v.b", L.b_in + L.c_vv, 1, G * dv, 0); }
       }
-      if (s.qk_norm && s.qk_norm != XOTB200_LM_QKNORM_HEAD_PLAIN) {
+      if (s.conv_taps > 0) {
+        const int C = H * dk + G * (dk + dv);
+        L.conv_ch = C;
+        L.conv_w = take((size_t)C * s.conv_taps);
+        dest(mp + "q.conv", L.conv_w, H * dk, s.conv_taps, 0);
+        dest(mp + "k.conv", L.conv_w, G * dk, s.conv_taps, H * dk);
+        dest(mp + "v.conv", L.conv_w, G * dv, s.conv_taps, (H + G) * dk);
+        L.conv_off = e->state_floats;
+        e->state_floats += (size_t)(s.conv_taps - 1) * C;
+      }
+      if (s.v_mix) {
+        L.vmix = take(1); dest(mp + "vmix", L.vmix, 1, 1, 0);
+        L.vmix_mode = li == v_first_layer ? 1 : 2;
+      }
+      if (s.qk_norm == XOTB200_LM_QKNORM_HEAD || s.qk_norm == XOTB200_LM_QKNORM_ROW) {
         const bool whole = s.qk_norm == XOTB200_LM_QKNORM_ROW;
         const int nq = whole ? H * dk : dk, nk = whole ? G * dk : dk;
         L.q_norm = take(nq); dest(mp + "q.norm", L.q_norm, 1, nq, 0);
         if (own) { L.k_norm = take(nk); dest(mp + "k.norm", L.k_norm, 1, nk, 0); }
       }
       if (s.out_bias) { L.o_b = take(D); dest(mp + "o.b", L.o_b, 1, D, 0); }
-      if (s.sink) { L.sink = take(H); dest(mp + "sink", L.sink, 1, H, 0); }
+      if (s.sink == XOTB200_LM_SINK_LEARNED) { L.sink = take(H); dest(mp + "sink", L.sink, 1, H, 0); }
       if (s.rel_buckets > 0) { L.rel = take((size_t)s.rel_buckets * H); dest(mp + "rel", L.rel, s.rel_buckets, H, 0); }
       if (s.dist_bias) {
         L.r1 = take(H); dest(mp + "r1", L.r1, 1, H, 0);
@@ -533,7 +579,7 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
     }
     e->max_in = std::max(e->max_in, L.ld_in);
     const bool has_ff = s.ff_kind == XOTB200_LM_FF_MOE ? s.experts > 0 : s.ff > 0;
-    if (has_ff) {
+    if (has_ff && !parallel) {
       L.norm2 = take(NW); dest(p + "norm2", L.norm2, 1, NW, 0);
       if (!post_rms && !pre_scalar) { L.norm2b = take(D); dest(p + "norm2" + nb, L.norm2b, 1, D, 0); }
       if (pre_scalar) sublayer_extras(L, p, 1);
@@ -578,9 +624,11 @@ static int build_layout(xotb200_lm* e, const xotb200_lm_layer* all) {
       e->max_eff = std::max(e->max_eff, F);
       e->max_experts = std::max(e->max_experts, E);
     } else if (has_ff) {
-      REQUIRE(s.ff_kind == XOTB200_LM_FF_RELU2 || s.ff_kind == XOTB200_LM_FF_XIELU || s.ff_kind == XOTB200_LM_FF_GELU || s.ff_kind == XOTB200_LM_FF_GELU_GATED,
+      REQUIRE(s.ff_kind == XOTB200_LM_FF_RELU2 || s.ff_kind == XOTB200_LM_FF_XIELU || s.ff_kind == XOTB200_LM_FF_GELU || s.ff_kind == XOTB200_LM_FF_GELU_GATED ||
+                  s.ff_kind == XOTB200_LM_FF_CLAMPED_GLU,
               "layer %d: unknown feed-forward kind %d", li, s.ff_kind);
-      if (s.ff_kind == XOTB200_LM_FF_GELU_GATED) {             // gate and up rows as one matrix (see glu_gate_row)
+      REQUIRE(s.ff_kind != XOTB200_LM_FF_CLAMPED_GLU || s.expert_limit > 0.f, "layer %d: the clamped feed-forward needs a positive limit", li);
+      if (s.ff_kind == XOTB200_LM_FF_GELU_GATED || s.ff_kind == XOTB200_LM_FF_CLAMPED_GLU) {             // gate and up rows as one matrix (see glu_gate_row)
         L.up = take((size_t)2 * s.ff * D);
         dest(p + "mlp.gate", L.up, s.ff, D, 0);
         dest(p + "mlp.up", L.up, s.ff, D, s.ff % 8 ? s.ff : 0);
@@ -643,7 +691,7 @@ static int upload_tensor(xotb200_lm* e, Dest& d, const void* host_bf16) {
 
 // does a tensor name belong to this shard? (so that an unknown name there is an error, and anything else is skipped)
 static bool owned_name(const xotb200_lm* e, const std::string& name) {
-  if (name == "embed" || name == "pos" || name == "embed.norm") return e->first;
+  if (name == "embed" || name == "pos" || name == "embed.norm" || name == "bigram") return e->first;
   if (name == "head" || name == "final.norm" || name == "final.norm.b" || name == "final.norm.alpha") return e->last;
   if (name.size() > 1 && name[0] == 'l' && isdigit((unsigned char)name[1])) {
     const int li = atoi(name.c_str() + 1);
@@ -794,10 +842,9 @@ static int ensure_scratch(xotb200_lm* e, int M, int n_want) {
     const size_t m = (size_t)std::max(M, 64), z = e->esz;
     TRY(regrow(e->x, m * D * 4 * (e->pre_scalar ? std::max(1, e->cfg.streams) : 1)));
     TRY(regrow(e->y, m * D * 4));
-    if (e->pre_scalar) {
-      TRY(regrow(e->y2, m * D * 4));
-      TRY(regrow(e->h0, m * D * 4));
-    }
+    if (e->pre_scalar || e->parallel) TRY(regrow(e->y2, m * D * 4));
+    if (e->pre_scalar) TRY(regrow(e->h0, m * D * 4));
+    TRY(regrow(e->vfirst, m * e->vfirst_n * 4));
     if (e->max_heads_rec) {
       TRY(regrow(e->gdec, m * e->max_heads_rec * 4));
       TRY(regrow(e->ginw, m * e->max_heads_rec * 4));
@@ -873,6 +920,7 @@ static int ensure_host_out(xotb200_lm* e, size_t floats) {
 struct StepPlan {
   int M = 0, n_seq = 0;
   const int *tokens = nullptr, *row_slot = nullptr, *row_pos = nullptr, *want = nullptr;   // device
+  const int* bigram_row = nullptr;                     // per row: its row of the hashed-pair table
   const Item* seqs = nullptr;
   std::map<int, std::pair<const Item*, int>> items;   // rows per attention work item -> (device list, count)
   // expanded prompt attention (bf16): per distinct window of the model's attention layers, the requests that bring many rows
@@ -1108,6 +1156,7 @@ static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout)
   const int slots = H + (own ? 2 * G : 0);
   bf16* q16 = sp.n_gqa_tiles > 0 ? static_cast<bf16*>(e->q16) : nullptr;
   const bool weighted = s.qk_norm == XOTB200_LM_QKNORM_HEAD || s.qk_norm == XOTB200_LM_QKNORM_ROW;
+  const bool rotated_norm = s.qk_norm == XOTB200_LM_QKNORM_HEAD_ROTATED;
   if (s.qk_norm == XOTB200_LM_QKNORM_ROW) {
     const int nt = std::min(1024, std::max(128, cdiv(H * dk, 4 * 32) * 32));
     auto pk = gqa_prepare_row_kernel<T>;
@@ -1116,6 +1165,30 @@ static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout)
     pk<<<M, nt, psm, e->stream>>>(e->proj, L.ld_in, L.c_q, L.c_kk, L.c_vv, s.proj_bias ? at<T>(e, L.b_in) : nullptr, at<T>(e, L.q_norm),
                                                         own ? at<T>(e, L.k_norm) : nullptr, e->cfg.norm_eps, H, G, dk, dv, own ? 1 : 0, s.q_temp_coef,
                                                         s.q_temp_every, sp.row_slot, sp.row_pos, pg, pool, e->qfull, q16);
+  } else if (s.conv_taps > 0 || rotated_norm || L.rot_mul != 1.f || L.vmix_mode) {
+    GqaPrep a{};
+    a.proj = e->proj; a.ld = L.ld_in; a.col_q = L.c_q; a.col_k = L.c_kk; a.col_v = L.c_vv;
+    a.bias = s.proj_bias ? at<T>(e, L.b_in) : nullptr;
+    a.conv_w = s.conv_taps > 0 ? at<T>(e, L.conv_w) : nullptr;
+    a.q_norm = weighted ? at<T>(e, L.q_norm) : nullptr;
+    a.k_norm = weighted ? at<T>(e, L.k_norm) : nullptr;
+    a.vmix = L.vmix_mode ? at<T>(e, L.vmix) : nullptr;
+    a.taps = s.conv_taps;
+    a.norm_when = s.qk_norm == XOTB200_LM_QKNORM_NONE ? 0 : rotated_norm ? 2 : 1;
+    a.eps = e->cfg.norm_eps;
+    a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.own_kv = own ? 1 : 0;
+    a.q_temp_coef = s.q_temp_coef; a.q_temp_every = s.q_temp_every;
+    a.freqs = s.rot_dims > 0 ? L.freqs : nullptr;
+    a.rot_dims = s.rot_dims; a.rot_layout = s.rot_layout; a.rot_mul = L.rot_mul;
+    a.state = e->state + L.conv_off; a.state_slot_stride = e->state_floats;
+    a.vfirst = e->vfirst; a.vmix_mode = L.vmix_mode;
+    // stretches of one row group each; as many heads per block as still leave a few blocks for every SM
+    const int zs = std::max(1, std::min(65535, cdiv(sp.max_rows, GQA_PREP_ROWS)));
+    a.spc = (int)std::max<long>(1, std::min<long>(8, (long)cdiv(M, GQA_PREP_ROWS) * slots / (8L * e->sm_count)));
+    const size_t psm = (size_t)GQA_PREP_ROWS * (dk + s.rot_dims) * 4;
+    auto pk = gqa_filter_prepare_kernel<T>;
+    TRY(opt_in_smem(pk, psm));
+    pk<<<dim3(sp.n_seq, cdiv(slots, a.spc), zs), 128, psm, e->stream>>>(a, sp.seqs, pg, pool, e->qfull, q16);
   } else {
     gqa_prepare_kernel<T><<<cdiv((long)M * slots, 8), 256, 0, e->stream>>>(
         e->proj, L.ld_in, L.c_q, L.c_kk, L.c_vv, s.proj_bias ? at<T>(e, L.b_in) : nullptr, weighted ? at<T>(e, L.q_norm) : nullptr,
@@ -1133,7 +1206,8 @@ static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout)
     e->launches++;
   }
   const GqaScore sc{s.scale, s.softcap, s.window, s.chunk, s.dist_bias ? at<T>(e, L.r1) : nullptr, s.dist_bias ? at<T>(e, L.r2) : nullptr,
-                    s.rel_buckets > 0 ? L.rel_tab : nullptr, L.rel_n, s.sink ? at<T>(e, L.sink) : nullptr, s.keep_first, s.pool, pool_rows};
+                    s.rel_buckets > 0 ? L.rel_tab : nullptr, L.rel_n, s.sink == XOTB200_LM_SINK_LEARNED ? at<T>(e, L.sink) : nullptr, s.keep_first, s.pool, pool_rows,
+                    s.sink == XOTB200_LM_SINK_ONE ? 1 : 0};
   const float* gate = s.out_gate ? e->proj : nullptr;
   const int qpi = gqa_rows_per_item(s);
   const auto& it = sp.items.at(-qpi);   // the lists of this mixer have negative keys
@@ -1160,8 +1234,7 @@ static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout)
     CK(cudaGetLastError());
     e->launches++;
     if (splits > 1) {
-      gqa_combine_kernel<T><<<dim3(it.second, cdiv(qpi * H, 8)), 256, 0, e->stream>>>(e->part, it.first, H, dv, splits, s.sink ? at<T>(e, L.sink) : nullptr, gate,
-                                                                                     s.out_gate, L.ld_in, L.c_g, static_cast<T*>(e->oh));
+      gqa_combine_kernel<T><<<dim3(it.second, cdiv(qpi * H, 8)), 256, 0, e->stream>>>(e->part, it.first, H, dv, splits, static_cast<const T*>(sc.sink), sc.sink_one, gate, s.out_gate, L.ld_in, L.c_g, static_cast<T*>(e->oh));
       CK(cudaGetLastError());
       e->launches++;
     }
@@ -1305,9 +1378,9 @@ static dim3 row_grid(const xotb200_lm* e, int M, int D, int threads) { return di
 
 static bool layer_has_ff(const xotb200_lm_layer& s) { return s.ff_kind == XOTB200_LM_FF_MOE ? s.experts > 0 : s.ff > 0; }
 
-// the feed-forward of a layer: h (T) -> y (fp32)
+// the feed-forward of a layer: h (T) -> yout (fp32)
 template <typename T>
-static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
+static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout) {
   const xotb200_lm_layer& s = L.s;
   const int D = e->cfg.width, M = sp.M;
   T* h = static_cast<T*>(e->h);
@@ -1328,7 +1401,7 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
     const int shared = Fs > 0 && !ride ? 1 : 0;
     if (shared) {
       TRY((product<T, T, T, 1>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, static_cast<T*>(e->act), s.shared_ff, 0, M, s.shared_ff, D, 1)));
-      TRY((product<T, T, float, 0>(e, static_cast<T*>(e->act), s.shared_ff, 0, at<T>(e, L.down), s.shared_ff, 1, 0, e->y, D, 0, M, D, s.shared_ff, 1)));
+      TRY((product<T, T, float, 0>(e, static_cast<T*>(e->act), s.shared_ff, 0, at<T>(e, L.down), s.shared_ff, 1, 0, yout, D, 0, M, D, s.shared_ff, 1)));
     }
     {
       // several rows per block when there are enough for all SMs and they fit in shared memory
@@ -1365,7 +1438,7 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
         if (r == 1) r = grouped_product<EPI_NONE, float>(e, ma, F, at<bf16>(e, L.w_edown), F, (long)D * F, E, e->moe_yg, D, m_pad, D, F, tile_expert);
         if (r < 0) return r;
         if (r == 1) {
-          moe_combine_kernel<bf16><<<row_grid(e, M, D, 256), 256, 0, e->stream>>>(e->moe_yg, place, e->moe_wts, top, D, shared, e->y, close);
+          moe_combine_kernel<bf16><<<row_grid(e, M, D, 256), 256, 0, e->stream>>>(e->moe_yg, place, e->moe_wts, top, D, shared, yout, close);
           CK(cudaGetLastError());
           e->launches++;
           e->closed = e->close != nullptr;
@@ -1387,7 +1460,7 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
       const size_t dsm = ((size_t)top * F + (ride ? Fs + 4 : 0)) * 4;
       TRY(opt_in_smem(kern, dsm));
       kern<<<dim3(M, std::max(1, std::min(cdiv(D, 16), M <= 16 ? 1024 : 16))), 256, dsm, e->stream>>>(static_cast<T*>(e->mact), F, at<T>(e, L.w_edown), D, e->moe_ids, e->moe_wts, top,
-                                                                                                   shared, e->y, static_cast<T*>(e->act), ride ? at<T>(e, L.down) : nullptr, Fs, close);
+                                                                                                   shared, yout, static_cast<T*>(e->act), ride ? at<T>(e, L.down) : nullptr, Fs, close);
       CK(cudaGetLastError());
       e->launches++;
       e->closed = e->close != nullptr;
@@ -1396,7 +1469,12 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
   }
   T* act = static_cast<T*>(e->act);
   EpiArgs epi;
-  if (s.ff_kind == XOTB200_LM_FF_GELU_GATED) {
+  if (s.ff_kind == XOTB200_LM_FF_CLAMPED_GLU) {
+    epi.il8 = s.ff % 8 == 0 ? 1 : 0;
+    epi.limit = s.expert_limit;
+    epi.slope = s.expert_slope;
+    TRY((product<T, T, T, EPI_CLAMPED_GLU>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, act, s.ff, 0, M, 2 * s.ff, D, 1, epi)));
+  } else if (s.ff_kind == XOTB200_LM_FF_GELU_GATED) {
     epi.il8 = s.ff % 8 == 0 ? 1 : 0;
     TRY((product<T, T, T, EPI_GELU_GLU>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, act, s.ff, 0, M, 2 * s.ff, D, 1, epi)));
   } else if (s.ff_kind == XOTB200_LM_FF_GELU) {
@@ -1407,7 +1485,7 @@ static int feed_forward(xotb200_lm* e, LmLayer& L, const StepPlan& sp) {
   } else {
     TRY((product<T, T, T, EPI_RELU2>(e, h, D, 0, at<T>(e, L.up), D, 1, 0, act, s.ff, 0, M, s.ff, D, 1)));
   }
-  return output_product<T>(e, act, L.down, s.ff, e->y, M);
+  return output_product<T>(e, act, L.down, s.ff, yout, M);
 }
 
 template <typename T>
@@ -1491,7 +1569,7 @@ static int run_layers_post(xotb200_lm* e, const StepPlan& sp, int n_want) {
     TRY(run_mixer<T>(e, L, sp));
     TRY(close(L.norm1, L.norm1b, L.s.mixer == XOTB200_LM_MIX_ATTENTION && L.s.out_bias ? at<T>(e, L.o_b) : nullptr));
     if (layer_has_ff(L.s)) {
-      TRY(feed_forward<T>(e, L, sp));
+      TRY(feed_forward<T>(e, L, sp, e->y));
       TRY(close(L.norm2, L.norm2b, nullptr));
     }
     if (e->trace) CK(cudaMemcpyAsync(e->trace_buf + li * (size_t)M * D, e->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, e->stream));
@@ -1562,7 +1640,7 @@ static int run_layers_pre_scalar(xotb200_lm* e, const StepPlan& sp, int n_want) 
     if (hc) { pend.mix = at<T>(e, L.hc_mix[0]); pend.out = at<T>(e, L.hc_out[0]); }
     if (layer_has_ff(L.s)) {
       TRY(open(&L, 1, nullptr));
-      TRY(feed_forward<T>(e, L, sp));
+      TRY(feed_forward<T>(e, L, sp, e->y));
       pend.y = e->y;
       if (hc) { pend.mix = at<T>(e, L.hc_mix[1]); pend.out = at<T>(e, L.hc_out[1]); }
     }
@@ -1627,7 +1705,7 @@ static int run_layers_pre_dyt(xotb200_lm* e, const StepPlan& sp, int n_want) {
     const LmLayer* after = li + 1 < e->layers.size() ? &e->layers[li + 1] : nullptr;
     const bool ff = layer_has_ff(L.s);
     TRY(sublayer([&]() { return run_mixer<T>(e, L, sp); }, L.ls1, ff ? &L : after, ff ? 1 : 0));
-    if (ff) TRY(sublayer([&]() { return feed_forward<T>(e, L, sp); }, L.ls2, after, 0));
+    if (ff) TRY(sublayer([&]() { return feed_forward<T>(e, L, sp, e->y); }, L.ls2, after, 0));
     if (e->trace) CK(cudaMemcpyAsync(e->trace_buf + li * (size_t)M * D, e->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, e->stream));
   }
   if (e->trace) e->trace_floats = e->layers.size() * (size_t)M * D;
@@ -1636,6 +1714,61 @@ static int run_layers_pre_dyt(xotb200_lm* e, const StepPlan& sp, int n_want) {
     dyt_rows_kernel<T><<<row_grid(e, n_want, D, nt), nt, 0, e->stream>>>(e->x, sp.want, at<T>(e, e->final_norm_a), at<T>(e, e->final_norm), at<T>(e, e->final_norm_b), hw, D);
     CK(cudaGetLastError());
     e->launches++;
+    TRY((product<T, T, float, EPI_NONE>(e, hw, D, 0, at<T>(e, e->head), D, 1, 0, e->logits, e->cfg.vocab, 0, n_want, e->cfg.vocab, D, 1)));
+    finish_logits(e, n_want);
+    CK(cudaGetLastError());
+  }
+  return 0;
+}
+
+// Parallel layers: h = rms(x) * w, x += mixer(h) + ff(h).  The two sublayers share nothing but h, so the feed-forward runs on the side stream
+// beside the mixer (in a captured decode step: two branches of the graph); one row pass adds both results and norms the sum for the next
+// layer.
+template <typename T>
+static int run_layers_parallel(xotb200_lm* e, const StepPlan& sp, int n_want) {
+  const int D = e->cfg.width, M = sp.M;
+  const float eps = e->cfg.norm_eps;
+  T* h = static_cast<T*>(e->h);
+  const int vec = D % 4 == 0 ? 4 : 1, nt = std::min(1024, std::max(64, cdiv(D, vec * 32) * 32));
+  auto kern = vec == 4 ? parallel_rows_kernel<T, 4> : parallel_rows_kernel<T, 1>;
+  TRY(opt_in_smem(kern, (size_t)D * 4));
+  const float *pend = nullptr, *pend2 = nullptr;
+  auto pass = [&](bool embed, const T* w, T* out, const int* rows, int n) -> int {
+    if (!embed && !pend && !w) return 0;
+    kern<<<n, nt, (size_t)D * 4, e->stream>>>(e->x, pend, pend2, embed ? at<T>(e, e->embed) : nullptr, sp.tokens, e->cfg.embed_scale != 0.f ? e->cfg.embed_scale : 1.0f,
+                                              e->cfg.bigram_buckets > 0 ? at<T>(e, e->bigram) : nullptr, sp.bigram_row, rows, w, eps, out, D);
+    CK(cudaGetLastError());
+    e->launches++;
+    if (!rows) pend = pend2 = nullptr;
+    return 0;
+  };
+  for (size_t li = 0; li < e->layers.size(); ++li) {
+    LmLayer& L = e->layers[li];
+    TRY(pass(e->first && li == 0, at<T>(e, L.norm1), h, nullptr, M));
+    const bool ff = layer_has_ff(L.s);
+    int rc = 0;
+    if (ff) {
+      CK(cudaEventRecord(e->ev_fork, e->stream));
+      CK(cudaStreamWaitEvent(e->side, e->ev_fork, 0));
+      std::swap(e->stream, e->side);
+      rc = feed_forward<T>(e, L, sp, e->y2);
+      std::swap(e->stream, e->side);
+    }
+    if (rc == 0) rc = run_mixer<T>(e, L, sp);
+    if (ff) {                                          // joined also after a failed launch: a capture must not end with the side stream still forked
+      const cudaError_t j1 = cudaEventRecord(e->ev_join, e->side), j2 = cudaStreamWaitEvent(e->stream, e->ev_join, 0);
+      if (rc >= 0) { CK(j1); CK(j2); }
+    }
+    if (rc < 0) return rc;
+    pend = e->y;
+    pend2 = ff ? e->y2 : nullptr;
+    if (e->trace || (!e->last && li + 1 == e->layers.size())) TRY(pass(false, nullptr, nullptr, nullptr, M));
+    if (e->trace) CK(cudaMemcpyAsync(e->trace_buf + li * (size_t)M * D, e->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, e->stream));
+  }
+  if (e->trace) e->trace_floats = e->layers.size() * (size_t)M * D;
+  if (e->last && n_want > 0) {
+    T* hw = static_cast<T*>(e->hw);
+    TRY(pass(false, at<T>(e, e->final_norm), hw, sp.want, n_want));
     TRY((product<T, T, float, EPI_NONE>(e, hw, D, 0, at<T>(e, e->head), D, 1, 0, e->logits, e->cfg.vocab, 0, n_want, e->cfg.vocab, D, 1)));
     finish_logits(e, n_want);
     CK(cudaGetLastError());
@@ -1653,6 +1786,7 @@ static int norm_threads(int D, int G) {
 template <typename T>
 static int run_layers(xotb200_lm* e, const StepPlan& sp, int n_want) {
   if (e->cfg.block == XOTB200_LM_BLOCK_PRE_SCALAR) return run_layers_pre_scalar<T>(e, sp, n_want);
+  if (e->cfg.block == XOTB200_LM_BLOCK_PARALLEL_RMS) return run_layers_parallel<T>(e, sp, n_want);
   if (e->cfg.block == XOTB200_LM_BLOCK_PRE_DYT) return run_layers_pre_dyt<T>(e, sp, n_want);
   if (e->cfg.block != XOTB200_LM_BLOCK_GROUP_RMS) return run_layers_post<T>(e, sp, n_want);
   const int D = e->cfg.width, G = e->cfg.norm_groups, M = sp.M;
@@ -1683,7 +1817,7 @@ static int run_layers(xotb200_lm* e, const StepPlan& sp, int n_want) {
     pend_w = at<T>(e, L.norm1b);
     if (layer_has_ff(L.s)) {
       TRY(open(at<T>(e, L.norm2)));
-      TRY(feed_forward<T>(e, L, sp));
+      TRY(feed_forward<T>(e, L, sp, e->y));
       pend_y = e->y;
       pend_w = at<T>(e, L.norm2b);
     }
@@ -1731,7 +1865,7 @@ int xotb200_lm_create(const xotb200_lm_cfg* cfg, const xotb200_lm_layer* layers,
   REQUIRE(cfg->width >= 1 && cfg->vocab >= 1, "width and vocab must be positive");
   REQUIRE(cfg->norm_groups >= 1 && cfg->width % cfg->norm_groups == 0, "width %d is not a multiple of norm_groups %d", cfg->width, cfg->norm_groups);
   REQUIRE(cfg->block == XOTB200_LM_BLOCK_GROUP_RMS || cfg->block == XOTB200_LM_BLOCK_POST_LN || cfg->block == XOTB200_LM_BLOCK_POST_RMS ||
-              cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR || cfg->block == XOTB200_LM_BLOCK_PRE_DYT,
+              cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR || cfg->block == XOTB200_LM_BLOCK_PRE_DYT || cfg->block == XOTB200_LM_BLOCK_PARALLEL_RMS,
           "unknown block form %d", cfg->block);
   REQUIRE(cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR || (cfg->streams == 0 && cfg->canon_taps == 0 && cfg->residual_mult == 0.f),
           "stream copies, input convolutions and a residual multiplier belong to the pre-norm block with one-number weights");
@@ -1741,8 +1875,12 @@ int xotb200_lm_create(const xotb200_lm_cfg* cfg, const xotb200_lm_layer* layers,
   REQUIRE(cfg->max_positions >= 0, "negative max_positions");
   REQUIRE(cfg->block != XOTB200_LM_BLOCK_GROUP_RMS || (!cfg->pos_sinusoid && !cfg->embed_norm),
           "a computed position vector and a norm on the embedding belong to the other block forms");
-  REQUIRE((cfg->block != XOTB200_LM_BLOCK_PRE_SCALAR && cfg->block != XOTB200_LM_BLOCK_PRE_DYT) || (!cfg->pos_sinusoid && cfg->max_positions == 0),
-          "the one-number and the Dynamic-Tanh pre-norm block forms add no position vector");
+  REQUIRE((cfg->block != XOTB200_LM_BLOCK_PRE_SCALAR && cfg->block != XOTB200_LM_BLOCK_PRE_DYT && cfg->block != XOTB200_LM_BLOCK_PARALLEL_RMS) ||
+              (!cfg->pos_sinusoid && cfg->max_positions == 0),
+          "the pre-norm block forms with one-number weights or a Dynamic Tanh and the parallel block form add no position vector");
+  REQUIRE(cfg->bigram_buckets >= 0 && cfg->bigram_mul_prev >= 0 && cfg->bigram_mul_cur >= 0, "negative size or factor of the hashed-pair table");
+  REQUIRE(cfg->block == XOTB200_LM_BLOCK_PARALLEL_RMS || (cfg->bigram_buckets == 0 && (cfg->embed_scale == 0.f || cfg->embed_scale == 1.f)),
+          "a scaled embedding and a hashed-pair table belong to the parallel block form");
   REQUIRE(cfg->block == XOTB200_LM_BLOCK_PRE_DYT || !cfg->layer_scale, "layer scales belong to the Dynamic-Tanh pre-norm block form");
   REQUIRE(!cfg->embed_norm || cfg->block == XOTB200_LM_BLOCK_POST_RMS || cfg->block == XOTB200_LM_BLOCK_PRE_SCALAR,
           "the norm on the embedding is the RMS norm of the post-RMS or the one-number pre-norm block form");
@@ -1784,7 +1922,14 @@ int xotb200_lm_create(const xotb200_lm_cfg* cfg, const xotb200_lm_layer* layers,
     std::vector<float> f(L.s.rot_dims / 2);
     for (int i = 0; i < L.s.rot_dims / 2; ++i) {
       double fi = pow((double)L.s.rot_base, -2.0 * i / L.s.rot_dims);
-      if (L.s.mixer == XOTB200_LM_MIX_ATTENTION && L.s.rot_scale_factor > 0.f) {
+      if (L.s.mixer == XOTB200_LM_MIX_ATTENTION && L.s.rot_scale_factor > 0.f && L.s.rot_scale_kind == XOTB200_LM_ROT_SCALE_YARN) {
+        const double n = L.s.rot_dims;
+        auto plane = [&](double turns) { return n * log((double)L.s.rot_scale_original / (2.0 * M_PI * turns)) / (2.0 * log((double)L.s.rot_base)); };
+        const double a = std::max(floor(plane(L.s.rot_scale_high)), 0.0), b = std::min(ceil(plane(L.s.rot_scale_low)), n - 1.0);
+        const double ramp = std::min(std::max((i - a) / std::max(b - a, 0.001), 0.0), 1.0);
+        fi = fi / L.s.rot_scale_factor * ramp + fi * (1.0 - ramp);
+        L.rot_mul = (float)(0.1 * log((double)L.s.rot_scale_factor) + 1.0);
+      } else if (L.s.mixer == XOTB200_LM_MIX_ATTENTION && L.s.rot_scale_factor > 0.f) {
         // long wavelengths are stretched by `factor`, short ones stay, the band between is blended by where the wavelength lies in it
         const double orig = L.s.rot_scale_original, lo = L.s.rot_scale_low, hi = L.s.rot_scale_high, fac = L.s.rot_scale_factor;
         const double wl = 2.0 * M_PI / fi;
@@ -1863,7 +2008,7 @@ int xotb200_lm_destroy(xotb200_lm* e) {
     if (L.rel_bucket) cudaFree(L.rel_bucket);
     if (L.rel_tab) cudaFree(L.rel_tab);
   }
-  void* ptrs[] = {e->oh2, e->y2, e->h0, e->gdec, e->ginw, e->gfloor, e->gnq, e->pos_freqs, e->dist_tab, e->moe_xg, e->moe_yg, e->moe_plan, e->dkk, e->drr, e->cvb, e->moe_ids, e->moe_wts, e->mact, e->du, e->dau, e->part, e->q16, e->cbuf, e->knx, e->vxx, e->blob, e->d_stage, e->x, e->y, e->proj, e->qraw, e->qfull, e->wlog, e->oraw, e->logits, e->h, e->cqn, e->qn, e->olat, e->oh, e->act,
+  void* ptrs[] = {e->vfirst, e->oh2, e->y2, e->h0, e->gdec, e->ginw, e->gfloor, e->gnq, e->pos_freqs, e->dist_tab, e->moe_xg, e->moe_yg, e->moe_plan, e->dkk, e->drr, e->cvb, e->moe_ids, e->moe_wts, e->mact, e->du, e->dau, e->part, e->q16, e->cbuf, e->knx, e->vxx, e->blob, e->d_stage, e->x, e->y, e->proj, e->qraw, e->qfull, e->wlog, e->oraw, e->logits, e->h, e->cqn, e->qn, e->olat, e->oh, e->act,
                   e->th, e->hw, e->d_argmax, e->trace_buf};
   for (void* p : ptrs)
     if (p) cudaFree(p);
@@ -1919,6 +2064,7 @@ int xotb200_lm_init_synthetic(xotb200_lm* e, uint64_t seed) {
     else if (ends(".A_log")) dev = 0.3f;
     else if (ends(".ls1") || ends(".ls2")) { mean = 0.5f; dev = 0.1f; }
     else if (ends(".correction")) dev = 0.1f;
+    else if (ends(".vmix")) { mean = 0.4f; dev = 0.1f; }
     else if (name.find("norm") != std::string::npos) { mean = 1.f; dev = 0.1f; }
     else if (d.rows == 1) dev = 0.5f;                  // biases of the delta-rule gates
     else if (name == "embed") dev = 1.f;
@@ -2042,6 +2188,7 @@ int xotb200_lm_begin(xotb200_lm* e, int max_tokens, int max_requests, int page_s
   e->free_pages.clear();
   for (int p = e->n_pages - 1; p >= 0; --p) e->free_pages.push_back(p);   // pages are handed out from the back: 0, 1, 2, ...
   e->slot_len.assign(max_requests, 0);
+  e->slot_last.assign(max_requests, 0);
   e->slot_pages.assign(max_requests, 0);
   CK(cudaStreamSynchronize(e->stream));
   return 0;
@@ -2114,7 +2261,9 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
       if (std::find(qpis.begin(), qpis.end(), q) == qpis.end()) qpis.push_back(q);
     }
   std::vector<int>& st = e->stage_build;
+  const bool bigram = e->first && e->cfg.bigram_buckets > 0;
   st.assign(3 * (size_t)M + n_want, 0);
+  std::vector<int> bg(bigram ? M : 0);
   std::vector<Item> seqs(n_seq);
   StepPlan sp;
   sp.M = (int)M;
@@ -2136,14 +2285,20 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
     sp.max_len = std::max(sp.max_len, len1);
     sp.max_rows = std::max(sp.max_rows, counts[i]);
     for (int t = 0; t < counts[i]; ++t, ++row) {
+      if (bigram) {
+        const int64_t B = e->cfg.bigram_buckets, prev = t > 0 ? tokens[row - 1] : e->slot_last[sl];
+        bg[row] = len0 + t == 0 ? (int)B : (int)((prev * (e->cfg.bigram_mul_prev % B) + tokens[row] * (e->cfg.bigram_mul_cur % B)) % B);
+      }
       st[row] = e->first ? tokens[row] : 0;
       st[M + row] = sl;
       st[2 * M + row] = len0 + t;
     }
   }
+  if (e->first)
+    for (int i = 0; i < n_seq; ++i) e->slot_last[slots[i]] = tokens[seqs[i].row0 + counts[i] - 1];
   for (int w = 0; w < n_want; ++w) st[3 * M + w] = want_rows[w];
   auto push = [&](const void* p, size_t n_ints) { const size_t o = st.size(); const int* q = static_cast<const int*>(p); st.insert(st.end(), q, q + n_ints); return o; };
-  const size_t off_seqs = push(seqs.data(), 4 * (size_t)n_seq);
+  const size_t off_seqs = push(seqs.data(), 4 * (size_t)n_seq), off_bigram = push(bg.data(), bg.size());
   auto is_long = [&](int i) { return use_flash && counts[i] >= FLASH_MIN_ROWS; };
   std::map<int, std::pair<size_t, int>> item_off;
   sp.any_short = false;
@@ -2209,7 +2364,7 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
   }
   memcpy(e->h_stage, st.data(), off * 4);
   if (e->last && n_want > 0) TRY(ensure_host_out(e, (size_t)n_want * V + n_want));
-  else if (!e->last) TRY(ensure_host_out(e, (size_t)M * D));
+  else if (!e->last) TRY(ensure_host_out(e, (size_t)M * (D + e->carry_out)));
   // Decoding — every request brings one row — has the same launches step after step: only the contents of the index arrays and
   // the lengths differ.  Such a step is captured into a CUDA graph the second time its shape is seen and replayed from then on.
   // What the launches depend on is in the key; the key length is a bucket of the longest request (it fixes how the absorbed
@@ -2248,6 +2403,7 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
       sp.row_slot = e->d_stage + M;
       sp.row_pos = e->d_stage + 2 * M;
       sp.want = e->d_stage + 3 * M;
+      sp.bigram_row = e->d_stage + off_bigram;
       sp.seqs = reinterpret_cast<const Item*>(e->d_stage + off_seqs);
       for (auto& kv : item_off) sp.items[kv.first] = {reinterpret_cast<const Item*>(e->d_stage + kv.second.first), kv.second.second};
       sp.gqa_tiles = reinterpret_cast<const GqaTile*>(e->d_stage + gqa_tiles_off);
@@ -2259,13 +2415,24 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
         f.n_reqs = kv.second.n_reqs; f.n_tiles = kv.second.n_tiles; f.n_keys = kv.second.n_keys; f.max_keys = kv.second.max_keys;
         sp.flash[kv.first] = f;
       }
-      if (!e->first) CK(cudaMemcpyAsync(e->x, hidden_f32, (size_t)M * D * 4, cudaMemcpyHostToDevice, e->stream));
+      // rows of the stream, each followed by the first mixing layer's values where those cross the border
+      auto copy_rows = [&](float* dst, size_t dld, const float* src, size_t sld, size_t n, cudaMemcpyKind kind) -> int {
+        CK(cudaMemcpy2DAsync(dst, dld * 4, src, sld * 4, n * 4, M, kind, e->stream));
+        return 0;
+      };
+      if (!e->first) {
+        const size_t ld = (size_t)D + e->carry_in;
+        TRY(copy_rows(e->x, D, hidden_f32, ld, D, cudaMemcpyHostToDevice));
+        if (e->carry_in) TRY(copy_rows(e->vfirst, e->carry_in, hidden_f32 + D, ld, e->carry_in, cudaMemcpyHostToDevice));
+      }
       TRY(e->esz == 2 ? run_layers<bf16>(e, sp, n_want) : run_layers<float>(e, sp, n_want));
       if (e->last && n_want > 0) {
         if (logits_f32) CK(cudaMemcpyAsync(e->h_out, e->logits, (size_t)n_want * V * 4, cudaMemcpyDeviceToHost, e->stream));
         if (argmax_i32) CK(cudaMemcpyAsync(e->h_out + (size_t)n_want * V, e->d_argmax, (size_t)n_want * 4, cudaMemcpyDeviceToHost, e->stream));
       } else if (!e->last) {
-        CK(cudaMemcpyAsync(e->h_out, e->x, (size_t)M * D * 4, cudaMemcpyDeviceToHost, e->stream));
+        const size_t ld = (size_t)D + e->carry_out;
+        TRY(copy_rows(e->h_out, ld, e->x, D, D, cudaMemcpyDeviceToHost));
+        if (e->carry_out) TRY(copy_rows(e->h_out + D, ld, e->vfirst, e->carry_out, e->carry_out, cudaMemcpyDeviceToHost));
       }
       CK(cudaMemcpyAsync(e->h_err, e->d_err, 4, cudaMemcpyDeviceToHost, e->stream));
       return 0;
@@ -2298,8 +2465,15 @@ int xotb200_lm_step(xotb200_lm* e, int n_seq, const int32_t* slots, const int32_
     if (logits_f32) memcpy(logits_f32, e->h_out, (size_t)n_want * V * 4);
     if (argmax_i32) memcpy(argmax_i32, e->h_out + (size_t)n_want * V, (size_t)n_want * 4);
   } else if (!e->last) {
-    memcpy(hidden_out_f32, e->h_out, (size_t)M * D * 4);
+    memcpy(hidden_out_f32, e->h_out, (size_t)M * (D + e->carry_out) * 4);
   }
+  return 0;
+}
+
+int xotb200_lm_hidden_width(xotb200_lm* e, int* in, int* out) {
+  REQUIRE(e && in && out, "null argument");
+  *in = e->first ? 0 : e->cfg.width + e->carry_in;
+  *out = e->last ? 0 : e->cfg.width + e->carry_out;
   return 0;
 }
 

@@ -2,7 +2,7 @@
 // reads the residual stream itself; a layer norm with weight and bias, or an RMS norm with a weight stored around zero, closes it),
 // with a learned position table or a computed sine/cosine position vector, short causal convolutions in front of a gated delta
 // rule, the two-sided xIELU activation and mixtures of experts (gated silu or relu^2 experts, two routing rules).
-// Also the pre-norm block form with a Dynamic Tanh norm (dyt_rows_kernel and the closing epilogue of layered_kernels.cuh), and the
+// Also the parallel block form (parallel_rows_kernel), the pre-norm block form with a Dynamic Tanh norm (dyt_rows_kernel and the closing epilogue of layered_kernels.cuh), and the
 // pre-norm block form whose norm weights are one number each: the stream kept in several copies mixed by
 // hyper-connections, and a causal convolution added to every sublayer input (embed_streams_kernel, hc_open_kernel, short_conv_kernel).
 //
@@ -137,6 +137,57 @@ __global__ void residual_rmsnorm_kernel(float* __restrict__ x, const float* __re
       x[(size_t)m * D + d] = v;
     }
     if (h) stf(h + (size_t)m * D + d, v);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------------
+// Row pass of the parallel block form (XOTB200_LM_BLOCK_PARALLEL_RMS): closes a layer and opens the next,
+//   t = x[m] + y[m] + y2[m]          (y, y2: the two sublayers' outputs; either may be NULL)
+//   t = embed[tokens[m]] * embed_scale + bigram[bigram_row[m]]           (embed != NULL: the start of the model; bigram may be NULL)
+//   h[m] = t / sqrt(mean(t^2) + eps) * w                                 (w == NULL: no norm follows)
+// and writes t back to x, unless src_rows names gathered rows (the final norm of the wanted rows: x, y, y2 are read at src_rows[m], h written
+// at m).  One block per row; VEC = 4: rows of whole 16-byte pieces.  Dynamic shared memory: D floats.
+// ---------------------------------------------------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void parallel_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ y2, const T* __restrict__ embed,
+                                     const int* __restrict__ tokens, float embed_scale, const T* __restrict__ bigram, const int* __restrict__ bigram_row,
+                                     const int* __restrict__ src_rows, const T* __restrict__ w, float eps, T* __restrict__ h, int D) {
+  extern __shared__ __align__(16) float par_row[];             // read back by the writing thread only
+  __shared__ float red[32];
+  const size_t m = blockIdx.x, src = src_rows ? src_rows[m] : m;
+  const T* er = embed ? embed + (size_t)tokens[m] * D : nullptr;
+  const T* br = embed && bigram ? bigram + (size_t)bigram_row[m] * D : nullptr;
+  const float *xr = x + src * D, *yr = y ? y + src * D : nullptr, *zr = y2 ? y2 + src * D : nullptr;
+  float ss = 0.f;
+  for (int d = threadIdx.x * VEC; d < D; d += blockDim.x * VEC) {
+    float v[VEC];
+    if (er) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = ldf(er + d + i) * embed_scale + (br ? ldf(br + d + i) : 0.f);
+    } else if constexpr (VEC == 4) {
+      const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 a = *reinterpret_cast<const float4*>(xr + d), b = yr ? *reinterpret_cast<const float4*>(yr + d) : z,
+                   c = zr ? *reinterpret_cast<const float4*>(zr + d) : z;
+      v[0] = a.x + (b.x + c.x); v[1] = a.y + (b.y + c.y); v[2] = a.z + (b.z + c.z); v[3] = a.w + (b.w + c.w);
+    } else {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = xr[d + i] + ((yr ? yr[d + i] : 0.f) + (zr ? zr[d + i] : 0.f));
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { ss = fmaf(v[i], v[i], ss); par_row[d + i] = v[i]; }
+    if (!src_rows && (er || yr || zr)) {
+      if constexpr (VEC == 4) *reinterpret_cast<float4*>(x + m * D + d) = make_float4(v[0], v[1], v[2], v[3]);
+      else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x[m * D + d + i] = v[i];
+      }
+    }
+  }
+  if (!w) return;
+  const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)D + eps);
+  for (int d = threadIdx.x * VEC; d < D; d += blockDim.x * VEC) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) stf(h + m * D + d + i, par_row[d + i] * r * ldf(w + d + i));
   }
 }
 

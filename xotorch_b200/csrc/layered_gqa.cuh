@@ -15,14 +15,14 @@
 //                 pool > 0: every block of `pool` tokens that ends at or before i - window is seen as ONE key / value, the means of
 //                 its cached keys / values (made by gqa_pool_blocks_kernel when the block's last token is appended; they live in
 //                 the second half of the layer's pool, block b of a request at the place token b has in the first half)
-//   weights     = softmax over the visible keys (fp32); with a sink the denominator also holds exp(sink[a]), a term that has no
-//                 key, no value, no scale and no bias and counts once; output = sum_j p_j v_j, times sigmoid(gate) per head or
+//   weights     = softmax over the visible keys (fp32); with a sink the denominator also holds exp(sink[a]) (sink_one: exp(0) = 1), a
+//                 term that has no key, no value, no scale and no bias and counts once; output = sum_j p_j v_j, times sigmoid(gate) per head or
 //                 per entry.
 // Queries and keys may be rotated by position before they are used / cached (first rot_dims entries of a head, fp32 angle).
 // Queries may carry a temperature: the query at position p is multiplied by 1 + coef * ln(1 + (p + 1) / every), integer quotient.
 //
 // Kernels: gqa_prepare_kernel (bias, per-head RMS norm, temperature, cache append), gqa_prepare_row_kernel (the same with ONE norm
-// over the whole query / key projection), gqa_attention_kernel + gqa_combine_kernel (one warp per (row, query head); decode,
+// over the whole query / key projection), gqa_filter_prepare_kernel (the same with short convolutions, norm after rotation, mixed values), gqa_attention_kernel + gqa_combine_kernel (one warp per (row, query head); decode,
 // short portions and the 32-bit mode), gqa_flash_kernel (tensor cores, bf16, long portions).
 #pragma once
 #include "layered_kernels.cuh"
@@ -41,7 +41,10 @@ struct GqaScore {
   int keep_first;    // > 0: the first tokens of a request that every later row sees
   int pool;          // > 0: tokens per pooled block
   size_t pool_rows;  // rows of the pool's first half (token rows); pooled block b of a request lives at pool_rows + row(slot, b)
+  int sink_one;      // 1: a sink of score 0 for every head (sink == NULL)
 };
+template <typename T>
+__device__ __forceinline__ float gqa_sink_score(const void* sink, int h) { return sink ? ldf(static_cast<const T*>(sink) + h) : 0.f; }
 
 // Keys a work item meets come in two stretches: `extra` keys in front (kept first tokens that lie before the item's token range, or
 // the pooled blocks its last row sees), then the tokens first .. last.  A VIRTUAL index v runs over both: v < extra -> extra key v.
@@ -189,6 +192,170 @@ __global__ void gqa_prepare_row_kernel(const float* __restrict__ proj, int ld, i
   }
 }
 
+// ---------------------------------------------------------------------------------------------------------------------------
+// The same step for layers with any of: short causal convolutions on the projections, a head norm AFTER the rotation, a rotation whose
+// cosines and sines carry a factor, values mixed with an earlier layer's.  In order, per row and channel:
+//   u = proj + bias;  f = sum_{j < taps} w[c, j] u(pos - taps + 1 + j)    (no filter when taps == 0; u of earlier steps from `state`)
+//   q, k: head norm (norm_when 1) -> rotation (times rot_mul) -> head norm (norm_when 2) -> query temperature -> qf / q16, pool
+//   v   : vmix_mode 1: f is also kept in vfirst [M, G * dv];  2: (1 - c) f + c vfirst, c = *vmix;  -> pool
+// grid (requests, groups of `spc` head slots, row stretches).  A stretch is at least taps - 1 rows, so only stretch 0 reads a slot's
+// filter inputs ([taps - 1][C] fp32 at `state`, zero at the start of a request) — and the threads that read a channel move its inputs on
+// after the last row they serve, in the same launch.  Rows go GQA_PREP_ROWS at a time: threads own channels and slide the filter down
+// the rows (a projection entry is loaded once per row group), the filtered heads wait in shared memory, then warps own rows.  The
+// rotation's cosines and sines of a row group are made once and serve all `spc` heads of the block.
+// Dynamic shared memory: GQA_PREP_ROWS * (dk + rot_dims) floats.
+// ---------------------------------------------------------------------------------------------------------------------------
+constexpr int GQA_PREP_ROWS = 8, GQA_PREP_TAPS = 8;   // rows per group; taps up to which weights and the sliding window stay in registers
+
+struct GqaPrep {
+  const float* proj;
+  int ld, col_q, col_k, col_v;
+  const void *bias, *conv_w, *q_norm, *k_norm, *vmix;   // T; NULL = none (bias is indexed by projection column, conv_w by channel: q | k | v)
+  int taps, norm_when;
+  float eps;
+  int H, G, dk, dv, own_kv, spc;
+  float q_temp_coef;
+  int q_temp_every;
+  const float* freqs;
+  int rot_dims, rot_layout;
+  float rot_mul;
+  float* state;
+  size_t state_slot_stride;
+  float* vfirst;
+  int vmix_mode;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128) gqa_filter_prepare_kernel(const GqaPrep a, const Item* __restrict__ seqs, Paging pg, T* __restrict__ pool, float* __restrict__ qf,
+                                                                 bf16* __restrict__ q16) {
+  extern __shared__ float prep_sm[];
+  float* fs = prep_sm;                                         // [GQA_PREP_ROWS][dk]: filtered entries of the head being prepared
+  float* cs = prep_sm + GQA_PREP_ROWS * a.dk;                  // [GQA_PREP_ROWS][rot_dims]: cosine, sine of every plane
+  const Item sq = seqs[blockIdx.x];
+  const int taps = max(a.taps, 1), keep = taps - 1, H = a.H, G = a.G, dk = a.dk, dv = a.dv;
+  const int C = H * dk + (a.own_kv ? G * (dk + dv) : 0), slots = H + (a.own_kv ? 2 * G : 0);
+  const int per = max((sq.n_rows + (int)gridDim.z - 1) / (int)gridDim.z, max(keep, 1));
+  const int t_begin = blockIdx.z * per, t_end = min(sq.n_rows, t_begin + per);
+  if (t_begin >= t_end) return;
+  const int s_begin = blockIdx.y * a.spc, s_end = min(slots, s_begin + a.spc);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T *bias = static_cast<const T*>(a.bias), *cw = static_cast<const T*>(a.conv_w);
+  float* st = keep > 0 ? a.state + (size_t)sq.slot * a.state_slot_stride : nullptr;
+  const int half = a.rot_dims >> 1;
+  const size_t rowlen = (size_t)G * (dk + dv);
+  const float vm = a.vmix_mode == 2 ? ldf(static_cast<const T*>(a.vmix)) : 0.f;
+  for (int t0 = t_begin; t0 < t_end; t0 += GQA_PREP_ROWS) {
+    const int n = min(GQA_PREP_ROWS, t_end - t0);
+    const bool last_group = t0 + n >= t_end;
+    if (a.freqs && s_begin < H + G)
+      for (int i = threadIdx.x; i < n * half; i += blockDim.x) {
+        float sn, cn;
+        sincosf((float)(sq.pos0 + t0 + i / half) * a.freqs[i % half], &sn, &cn);
+        cs[2 * i] = cn * a.rot_mul;
+        cs[2 * i + 1] = sn * a.rot_mul;
+      }
+    for (int sl = s_begin; sl < s_end; ++sl) {
+      const bool is_q = sl < H, is_v = sl >= H + G;
+      const int hd = is_q ? sl : is_v ? sl - H - G : sl - H, dim = is_v ? dv : dk;
+      const int c0 = (is_q ? a.col_q : is_v ? a.col_v : a.col_k) + hd * dim;      // projection column of the head's first channel
+      // ---- filter: one thread per channel
+      for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+        const int col = c0 + d, ch = col - a.col_q;
+        const float b = bias ? ldf(bias + col) : 0.f;
+        const float* pr = a.proj + (size_t)sq.row0 * a.ld + col;
+        auto input = [&](int r) { return r >= 0 ? pr[(size_t)r * a.ld] + b : st[(size_t)(r + keep) * C + ch]; };   // row r of this step
+        auto put = [&](int r, float f) {
+          if (!is_v) { fs[(r - t0) * dk + d] = f; return; }
+          const size_t m = sq.row0 + r;
+          float* vf = a.vmix_mode ? a.vfirst + m * (size_t)(G * dv) + hd * dv + d : nullptr;
+          if (a.vmix_mode == 1) *vf = f;
+          if (a.vmix_mode == 2) f = (1.0f - vm) * f + vm * *vf;
+          stf(pool + pg.row(sq.slot, sq.pos0 + r) * rowlen + (size_t)G * dk + hd * dv + d, f);
+        };
+        if (!cw) {
+          for (int r = t0; r < t0 + n; ++r) put(r, input(r));
+        } else if (taps <= GQA_PREP_TAPS) {
+          float wr[GQA_PREP_TAPS], win[GQA_PREP_TAPS], cur[GQA_PREP_ROWS];
+#pragma unroll
+          for (int i = 0; i < GQA_PREP_ROWS; ++i) cur[i] = i < n ? pr[(size_t)(t0 + i) * a.ld] + b : 0.f;
+#pragma unroll
+          for (int i = 0; i < GQA_PREP_TAPS; ++i) {
+            wr[i] = i < taps ? ldf(cw + (size_t)ch * taps + i) : 0.f;
+            win[i] = i < keep ? input(t0 - keep + i) : 0.f;
+          }
+#pragma unroll
+          for (int r = 0; r < GQA_PREP_ROWS; ++r) {
+            if (r >= n) break;
+            float f = 0.f;
+#pragma unroll
+            for (int i = 0; i < GQA_PREP_TAPS; ++i) {
+              if (i == keep) win[i] = cur[r];
+              if (i < taps) f = fmaf(wr[i], win[i], f);
+            }
+#pragma unroll
+            for (int i = 0; i + 1 < GQA_PREP_TAPS; ++i) win[i] = win[i + 1];
+            put(t0 + r, f);
+          }
+        } else {
+          for (int r = t0; r < t0 + n; ++r) {
+            float f = 0.f;
+            for (int i = 0; i < taps; ++i) f = fmaf(ldf(cw + (size_t)ch * taps + i), input(r - keep + i), f);
+            put(r, f);
+          }
+        }
+        if (blockIdx.z == 0 && last_group)
+          for (int i = 0; i < keep; ++i) {                     // increasing i: entry i + n_rows is still the old one when it is read
+            const int r = sq.n_rows - keep + i;
+            st[(size_t)i * C + ch] = r >= 0 ? pr[(size_t)r * a.ld] + b : st[(size_t)(i + sq.n_rows) * C + ch];
+          }
+      }
+      if (is_v) continue;
+      __syncthreads();
+      // ---- norm, rotation, norm: one warp per row
+      for (int r = warp; r < n; r += 4) {
+        float* f = fs + r * dk;
+        const float* c2 = cs + (size_t)r * a.rot_dims;
+        const T* w = static_cast<const T*>(is_q ? a.q_norm : a.k_norm);
+        const int pos = sq.pos0 + t0 + r;
+        float fac = is_q ? gqa_query_temperature(a.q_temp_coef, a.q_temp_every, pos) : 1.0f;
+        if (a.norm_when == 1) {
+          float ss = 0.f;
+          for (int d = lane; d < dk; d += 32) ss = fmaf(f[d], f[d], ss);
+          const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)dk + a.eps);
+          for (int d = lane; d < dk; d += 32) f[d] *= rs * (w ? ldf(w + d) : 1.f);
+          __syncwarp();
+        }
+        if (a.freqs) {
+          for (int i = lane; i < half; i += 32) {
+            const int du = a.rot_layout ? i : 2 * i, dw = a.rot_layout ? i + half : 2 * i + 1;
+            const float u = f[du], v = f[dw], cn = c2[2 * i], sn = c2[2 * i + 1];
+            f[du] = u * cn - v * sn;
+            f[dw] = v * cn + u * sn;
+          }
+          __syncwarp();
+        }
+        if (a.norm_when == 2) {
+          float ss = 0.f;
+          for (int d = lane; d < dk; d += 32) ss = fmaf(f[d], f[d], ss);
+          fac *= 1.0f / sqrtf(warp_sum(ss) / (float)dk + a.eps);
+        }
+        if (is_q) {
+          const size_t o = ((size_t)(sq.row0 + t0 + r) * H + hd) * dk;
+          for (int d = lane; d < dk; d += 32) {
+            const float v = f[d] * fac * (a.norm_when == 2 && w ? ldf(w + d) : 1.f);
+            qf[o + d] = v;
+            if (q16) q16[o + d] = __float2bfloat16_rn(v);
+          }
+        } else {
+          T* dst = pool + pg.row(sq.slot, pos) * rowlen + (size_t)hd * dk;
+          for (int d = lane; d < dk; d += 32) stf(dst + d, f[d] * fac * (a.norm_when == 2 && w ? ldf(w + d) : 1.f));
+        }
+      }
+      __syncthreads();                                         // the next head overwrites fs
+    }
+  }
+}
+
 // table[a][d] = rel[bucket_of[d], a] for d < n: the learned bias of head a at distance d (rel is [buckets, H] as stored)
 template <typename T>
 __global__ void gqa_rel_table_kernel(const T* __restrict__ rel, const int* __restrict__ bucket_of, int H, int n, float* __restrict__ table) {
@@ -323,7 +490,7 @@ __global__ void gqa_attention_kernel(const float* __restrict__ qf, const T* __re
     }
     return;
   }
-  const float corr = sc.sink ? apply_sink(ldf(static_cast<const T*>(sc.sink) + h), mx, den) : 1.0f;
+  const float corr = sc.sink || sc.sink_one ? apply_sink(gqa_sink_score<T>(sc.sink, h), mx, den) : 1.0f;
   const float inv = corr / den;
   T* o = out + (size_t)m * H * dv + (size_t)h * dv;
 #pragma unroll
@@ -333,11 +500,11 @@ __global__ void gqa_attention_kernel(const float* __restrict__ qf, const T* __re
   }
 }
 
-// merges the key runs: one warp per (row, query head) of the listed items; at most 32 runs.  A sink (per head, may be NULL) joins
-// here, once, like a run that holds the weight exp(sink) and no values.
+// merges the key runs: one warp per (row, query head) of the listed items; at most 32 runs.  A sink (per head, or of score 0 for all with
+// sink_one) joins here, once, like a run that holds the weight exp(sink) and no values.
 template <typename T>
 __global__ void gqa_combine_kernel(const float* __restrict__ part, const Item* __restrict__ items, int H, int dv, int splits, const T* __restrict__ sink,
-                                   const float* __restrict__ gate, int gate_mode, int gate_ld, int gate_col0, T* __restrict__ out) {
+                                   int sink_one, const float* __restrict__ gate, int gate_mode, int gate_ld, int gate_col0, T* __restrict__ out) {
   const Item it = items[blockIdx.x];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int pair = blockIdx.y * nw + warp;
@@ -345,10 +512,10 @@ __global__ void gqa_combine_kernel(const float* __restrict__ part, const Item* _
   const int m = it.row0 + pair / H, h = pair % H;
   const float* src = part + ((size_t)m * H + h) * splits * (size_t)(2 + dv);
   const float mz = lane < splits ? src[(size_t)lane * (2 + dv)] : -INFINITY;
-  const float sk = sink ? ldf(sink + h) : -INFINITY;
+  const float sk = sink || sink_one ? gqa_sink_score<T>(sink, h) : -INFINITY;
   const float mx = fmaxf(warp_max(mz), sk);
   const float wz = mz == -INFINITY ? 0.f : expf(mz - mx);
-  const float den = warp_sum(lane < splits ? src[(size_t)lane * (2 + dv) + 1] * wz : 0.f) + (sink ? expf(sk - mx) : 0.f);
+  const float den = warp_sum(lane < splits ? src[(size_t)lane * (2 + dv) + 1] * wz : 0.f) + (sink || sink_one ? expf(sk - mx) : 0.f);
   const float inv = 1.0f / den;
   for (int d0 = 0; d0 < dv; d0 += 32) {
     const int d = d0 + lane;
@@ -560,7 +727,7 @@ gqa_flash_kernel(const bf16* __restrict__ q16, const bf16* __restrict__ pool, Pa
     const int qi = warp * 16 + gq + r * 8;
     if (qi >= tl.n_rows) continue;
     const size_t m = tl.row0 + qi;
-    const float corr = sc.sink ? apply_sink(__bfloat162float(static_cast<const bf16*>(sc.sink)[h]), mx[r], den[r]) : 1.0f;
+    const float corr = sc.sink || sc.sink_one ? apply_sink(gqa_sink_score<bf16>(sc.sink, h), mx[r], den[r]) : 1.0f;
     const float inv = corr / den[r];
     bf16* dst = out + m * ((size_t)H * dv) + (size_t)h * dv;
 #pragma unroll

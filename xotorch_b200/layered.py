@@ -90,6 +90,8 @@ class LayerSpec:
   router_correction: int = 0
   group_best: int = 0
   router_scale: float = 0.0
+  rot_scale_kind: int = 0
+  v_mix: int = 0
 
   def to_c(self) -> LmLayer:
     c = LmLayer()
@@ -384,9 +386,63 @@ def rinutar_globals(config: dict) -> dict:
               block=_lib.LM_BLOCK_PRE_DYT, layer_scale=1, tied_head=1)
 
 
+# ---- the Fekanex family ------------------------------------------------------------------------------------------------------
+# config.json: {"architecture": "Fekanex", "width", "vocab", "norm": {"eps"}, "logit_scale", "embedding": {"scale", "bigram": {"buckets",
+#               "mul_prev", "mul_cur"}}, "layers": [{"type", "mixer", "mlp"}]}
+# A layer is parallel: h = rms(x) * w, x += mixer(h) + ff(h).  The embedding is scaled and a hashed (previous token, token) row is added;
+# the logits use the embedding table without the scale, times logit_scale.
+#   type "attention"  grouped-query attention (mixer: heads, kv_heads, dim, vdim, scale, conv = taps, rot {base, dims, scaling {factor,
+#                     original, fast, slow}}, mask {size, keep_first}, v_mix): biased projections through short causal convolutions, pairs
+#                     (2i, 2i + 1) rotated (YaRN frequencies), weightless RMS norm of every rotated query / key head, sliding window that
+#                     keeps the first tokens, a sink of score 0, values mixed with those of the first v_mix layer
+#   mlp.kind "dense"  clamped gated (mlp.ff, mlp.limit);  "moe": gated silu experts (mlp.expert.ff), the `top` largest router logits,
+#                     softmax over them (mlp.router {experts, top})
+FEKANEX_GLU_SLOPE = 1.702
+
+
+def _fekanex_ff(i: int, mlp) -> dict:
+  if mlp is None:
+    return dict(ff=0, ff_kind=_lib.LM_FF_CLAMPED_GLU)
+  kind = mlp.get("kind", "dense")
+  if kind == "dense":
+    return dict(ff=int(mlp["ff"]), ff_kind=_lib.LM_FF_CLAMPED_GLU, expert_limit=float(mlp["limit"]), expert_slope=FEKANEX_GLU_SLOPE)
+  if kind == "moe":
+    r = mlp["router"]
+    return dict(ff=0, ff_kind=_lib.LM_FF_MOE, experts=int(r["experts"]), top=int(r["top"]), expert_ff=int(mlp["expert"]["ff"]),
+                expert_act=_lib.LM_EXPERT_SILU_GATED, router_kind=_lib.LM_ROUTER_TOPK_SOFTMAX)
+  raise ValueError(f"layer {i}: feed-forward kind {kind!r} is not implemented (dense, moe)")
+
+
+def fekanex_layers(config: dict, shapes: Dict[str, Tuple[int, ...]]) -> List[LayerSpec]:
+  out = []
+  for i, layer in enumerate(config["layers"]):
+    kind, m = layer["type"], layer["mixer"]
+    if kind != "attention":
+      raise ValueError(f"layer {i}: mixer type {kind!r} is not implemented")
+    mask, rot = m.get("mask") or {}, m.get("rot") or {}
+    sc = rot.get("scaling") or {}
+    window = int(mask.get("size") or 0)
+    yarn = dict(rot_scale_kind=_lib.LM_ROT_SCALE_YARN, rot_scale_factor=float(sc["factor"]), rot_scale_original=float(sc["original"]),
+                rot_scale_high=float(sc["fast"]), rot_scale_low=float(sc["slow"])) if sc else {}
+    out.append(LayerSpec(
+      mixer=_lib.LM_MIX_ATTENTION, heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=int(m["dim"]), vdim=int(m["vdim"]),
+      scale=float(m["scale"]), window=window, keep_first=int(mask.get("keep_first") or 0) if window else 0, rot_dims=int(rot.get("dims", 0)),
+      rot_base=float(rot.get("base", 10000.0)), rot_layout=_lib.LM_ROT_INTERLEAVED, qk_norm=_lib.LM_QKNORM_HEAD_ROTATED, proj_bias=1,
+      conv_taps=int(m.get("conv") or 0), sink=_lib.LM_SINK_ONE, v_mix=1 if m.get("v_mix") else 0, **yarn, **_fekanex_ff(i, layer.get("mlp"))))
+  return out
+
+
+def fekanex_globals(config: dict) -> dict:
+  emb = config.get("embedding") or {}
+  bg = emb.get("bigram") or {}
+  return dict(width=int(config["width"]), vocab=int(config["vocab"]), norm_groups=1, norm_eps=float(config["norm"]["eps"]),
+              block=_lib.LM_BLOCK_PARALLEL_RMS, tied_head=1, embed_scale=float(emb.get("scale", 1.0)), logit_scale=float(config.get("logit_scale", 1.0)),
+              bigram_buckets=int(bg.get("buckets", 0)), bigram_mul_prev=int(bg.get("mul_prev", 0)), bigram_mul_cur=int(bg.get("mul_cur", 0)))
+
+
 LAYERED_FAMILIES = {"Zokuvik": (zokuvik_layers, zokuvik_globals), "Bufulorn": (bufulorn_layers, bufulorn_globals),
                     "Tunavik": (tunavik_layers, tunavik_globals), "Fubelorn": (fubelorn_layers, fubelorn_globals),
-                    "Rinutar": (rinutar_layers, rinutar_globals)}
+                    "Rinutar": (rinutar_layers, rinutar_globals), "Fekanex": (fekanex_layers, fekanex_globals)}
 
 
 class LayeredShard:
@@ -447,11 +503,16 @@ class LayeredShard:
     cfg.streams, cfg.canon_taps = self.globals.get("streams", 0), self.globals.get("canon_taps", 0)
     cfg.residual_mult = self.globals.get("residual_mult", 0.0)
     cfg.layer_scale, cfg.tied_head = self.globals.get("layer_scale", 0), self.globals.get("tied_head", 0)
+    cfg.embed_scale, cfg.bigram_buckets = self.globals.get("embed_scale", 0.0), self.globals.get("bigram_buckets", 0)
+    cfg.bigram_mul_prev, cfg.bigram_mul_cur = self.globals.get("bigram_mul_prev", 0), self.globals.get("bigram_mul_cur", 0)
     cfg.dtype = _lib.LM_DTYPE_F32 if self.dtype == "float32" else _lib.LM_DTYPE_BF16
     arr = (LmLayer * len(specs))(*[s.to_c() for s in specs])
     h = C.c_void_p()
     check_lm(self.lib.xotb200_lm_create(C.byref(cfg), arr, self.device, C.byref(h)))
     self.h, self.specs = h, specs
+    w_in, w_out = C.c_int(), C.c_int()
+    check_lm(self.lib.xotb200_lm_hidden_width(h, C.byref(w_in), C.byref(w_out)))
+    self.hidden_in, self.hidden_out = int(w_in.value), int(w_out.value)
     self.start, self.end = int(start_layer), int(end_layer)
     self.n_slots = 0
 
@@ -503,8 +564,8 @@ class LayeredShard:
   def step(self, slots: Sequence[int], rows: Sequence[np.ndarray], want: Optional[Sequence[int]] = None, logits: bool = True,
            argmax: bool = True):
     """One batched step.  rows[i]: the next token ids (1-D int) of slot slots[i] on the first shard, else its hidden state
-    [n_i, width] float32.  want: packed row indices whose output is asked for (default: every request's last row).
-    Last shard -> (logits [n_want, vocab] float32 | None, argmax [n_want] int32 | None); other shards -> hidden [sum n_i, width]."""
+    [n_i, hidden_in] float32 (the stream, `width` floats, and whatever else an earlier shard hands over: see xotb200_lm_hidden_width).  want: packed row indices whose output is asked for (default: every request's last row).
+    Last shard -> (logits [n_want, vocab] float32 | None, argmax [n_want] int32 | None); other shards -> hidden [sum n_i, hidden_out]."""
     n_seq = len(slots)
     if self.is_first:
       parts = [np.ascontiguousarray(r, dtype=np.int32).reshape(-1) for r in rows]
@@ -512,7 +573,7 @@ class LayeredShard:
       tok = np.ascontiguousarray(np.concatenate(parts)) if parts else np.zeros(0, np.int32)
       tok_p, hid_p = tok.ctypes.data_as(C.c_void_p), None
     else:
-      parts = [np.ascontiguousarray(r, dtype=np.float32).reshape(-1, self.width) for r in rows]
+      parts = [np.ascontiguousarray(r, dtype=np.float32).reshape(-1, self.hidden_in) for r in rows]
       counts = np.array([p.shape[0] for p in parts], dtype=np.int32)
       hid = np.ascontiguousarray(np.concatenate(parts, axis=0))
       tok_p, hid_p = None, hid.ctypes.data_as(C.c_void_p)
@@ -526,7 +587,7 @@ class LayeredShard:
       lg = np.empty((wn.size, self.vocab), dtype=np.float32) if logits else None
       am = np.empty(wn.size, dtype=np.int32) if argmax else None
     else:
-      ho = np.empty((M, self.width), dtype=np.float32)
+      ho = np.empty((M, self.hidden_out), dtype=np.float32)
     p = lambda a: a.ctypes.data_as(C.c_void_p) if a is not None else None
     check_lm(self.lib.xotb200_lm_step(self.h, n_seq, p(sl), p(counts), tok_p, hid_p, p(wn), int(wn.size) if self.is_last else 0, p(lg), p(am), p(ho)))
     if self.is_last:
@@ -549,7 +610,7 @@ class LayeredShard:
     if self.is_last:
       self._last_token = int(out[1][0])
       return out[0].reshape(1, -1)
-    return out.reshape(1, -1, self.width)
+    return out.reshape(1, -1, self.hidden_out)
 
   def last_token(self) -> int:
     if self._last_token is None:
