@@ -87,7 +87,8 @@ def softmax_one_more(scores: Tensor) -> Tensor:
 
 
 def projected(h: Tensor, W: Dict[str, Tensor], name: str) -> Tensor:
-  return causal_filter(h @ W[name].T + W[name + ".b"], W[name + ".conv"])
+  u = h @ W[name].T + W[name + ".b"]
+  return causal_filter(u, W[name + ".conv"]) if name + ".conv" in W else u
 
 
 def attention(h: Tensor, W: Dict[str, Tensor], m: dict, eps: float, first_values: Optional[Tensor]) -> Tuple[Tensor, Tensor]:
@@ -169,7 +170,9 @@ def tensor_shapes(cfg: dict) -> Dict[str, Tuple[int, ...]]:
     p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
     out[p + "norm1"] = (D,)
     for name, n in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
-      out.update({p + f"mix.{name}": (n, D), p + f"mix.{name}.b": (n,), p + f"mix.{name}.conv": (n, m["conv"])})
+      out.update({p + f"mix.{name}": (n, D), p + f"mix.{name}.b": (n,)})
+      if m.get("conv"):
+        out[p + f"mix.{name}.conv"] = (n, m["conv"])
     out[p + "mix.o"] = (D, m["heads"] * m["vdim"])
     if m.get("v_mix"):
       out[p + "mix.vmix"] = ()

@@ -20,6 +20,11 @@ clamped gated experts in turn) beside the two closest existing families on the s
 dense feed-forwards (as many weight bytes as a Rinutar token touches), and a Bufulorn model with the same alternation of dense and expert
 feed-forwards (to a few per cent the same weight bytes).
 
+`--layered-family fekanex`: the same for Fekanex-shaped models (parallel layers; grouped-query attention with short convolutions, rotation,
+mixed values, a window that keeps the first tokens; clamped gated feed-forwards and gated experts in turn) beside the closest existing family
+on the same engine, a Bufulorn model of attention layers with the same heads and the same alternation of dense and expert feed-forwards, of
+(to a few per cent) the same weight bytes.
+
 Timing: every number is the device time of the step(s) (CUDA events on the engine's stream, `last_step_ms` / the ring's own
 timer), after warm-up; the weights of every size are larger than L2 from `medium` on, and each prompt step streams all of them.
 Roofline denominators come from MEASURED_PEAKS.json (fallback: the profiling recipe's numbers)."""
@@ -198,12 +203,29 @@ def zokuvik_attention_config(s: dict):
 
 
 def bufulorn_alternating_config(s: dict, b: dict, context: int):
-  """Bufulorn attention layers whose feed-forwards are dense (xIELU, two matrices of the bytes of Rinutar's three) and experts in turn"""
+  """Bufulorn attention layers whose feed-forwards are dense (xIELU, two matrices of the bytes of a gated form's three) and experts in turn"""
   m = {"heads": b["heads"], "kv_heads": b["kv_heads"], "dim": b["dim"], "vdim": b["vdim"], "scale": float(b["dim"] ** -0.5), "softcap": 30.0}
   dense = {"kind": "dense", "ff": s["ff"] * 3 // 2}
   moe = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP, "groups": {"count": GROUPS, "keep": KEEP}}, "expert": {"ff": s["ff"] // 4}}
   layers = [{"type": "attention", "mixer": m, "mlp": mlp} for _ in range(3 * s["repeats"] // 2) for mlp in (dense, moe)]
   cfg = {"architecture": "Bufulorn", "width": s["width"], "vocab": s["vocab"], "max_positions": context, "norm": {"eps": 1e-5}, "layers": layers}
+  return cfg, len(layers) // 2 * (EXPERTS - TOP) * 3 * (s["ff"] // 4) * s["width"] * 2
+
+
+# Fekanex shapes at the same widths: attention heads as the Bufulorn attention layers (half of every head rotated), window 1024 keeping 4 tokens, six
+# layers with dense clamped gated feed-forwards and experts (16 of a quarter of the dense inner size, 4 per token) in turn
+FEK_KEEP, FEK_BUCKETS = 4, 65521
+
+
+def fekanex_config(s: dict, b: dict):
+  mixer = {"heads": b["heads"], "kv_heads": b["kv_heads"], "dim": b["dim"], "vdim": b["vdim"], "conv": TAPS, "scale": float(b["dim"] ** -0.5), "v_mix": True,
+           "mask": {"size": WINDOW, "keep_first": FEK_KEEP},
+           "rot": {"base": 500000.0, "dims": b["dim"] // 2, "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+  dense = {"kind": "dense", "ff": s["ff"], "limit": 7.0}
+  moe = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP}, "expert": {"ff": s["ff"] // 4}}
+  layers = [{"type": "attention", "mixer": mixer, "mlp": mlp} for _ in range(3 * s["repeats"] // 2) for mlp in (dense, moe)]
+  cfg = {"architecture": "Fekanex", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+         "embedding": {"scale": 2.0, "bigram": {"buckets": FEK_BUCKETS, "mul_prev": 10007, "mul_cur": 31}}, "layers": layers}
   return cfg, len(layers) // 2 * (EXPERTS - TOP) * 3 * (s["ff"] // 4) * s["width"] * 2
 
 
@@ -229,7 +251,7 @@ def layered_numbers(s: dict, prompts, decode_ctx: int, decode_batches, steps: in
   wbytes = eng.weight_bytes()
   # a prompt step streams the body once + one row of the embedding (and of the position table) per token
   tables = 1 if eng.globals.get("tied_head") else 2                      # embedding and head
-  body = wbytes - tables * 2 * s["vocab"] * s["width"] - int(cfg.get("max_positions", 0)) * s["width"] * 2 - idle_bytes
+  body = wbytes - (tables * s["vocab"] + int(eng.globals.get("bigram_buckets", 0))) * 2 * s["width"] - int(cfg.get("max_positions", 0)) * s["width"] * 2 - idle_bytes
   rng = np.random.default_rng(0)
   out = {"weight_bytes": wbytes, "prefill": {}, "decode": {}}
   max_b = max(decode_batches)
@@ -413,6 +435,22 @@ def run_rinutar(args, sizes, prompts, hbm, tf, src) -> None:
     print(json.dumps(line), flush=True)
 
 
+def run_fekanex(args, sizes, prompts, hbm, tf, src) -> None:
+  for name in sizes:
+    s, b = SIZES[name], BUFULORN[name]
+    warm = max(3, args.warmup)
+    context = max(max(prompts), 1024 + 9 * (args.steps * 8 + warm)) + 64
+    cfg, idle = fekanex_config(s, b)
+    bcfg, bidle = bufulorn_alternating_config(s, b, context)
+    models = {"fekanex": (cfg, idle), "bufulorn_same_size": (bcfg, bidle)}
+    out = {k: layered_numbers(s, prompts, decode_ctx=1024, decode_batches=[1, 8], steps=args.steps, warmup=warm, cfg=c, idle_bytes=i) for k, (c, i) in models.items()}
+    line = {"bench": "layered", "family": "fekanex", "size": name, "dtype": "bf16", "data": "synthetic", "shape": dict(s, **b), "idle_expert_bytes": idle, **out,
+            "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
+            "frac_of_peak": {**{f"{k}_decode1_hbm": round(v["decode"]["1"]["gbs_weights_device"] / hbm, 3) for k, v in out.items()},
+                             **{f"{k}_prefill{n}_tensor": round(v["prefill"][str(n)]["tflops_weights"] / tf, 3) for k, v in out.items() for n in prompts}}}
+    print(json.dumps(line), flush=True)
+
+
 def run(args) -> None:
   hbm, tf, src = peaks()
   sizes = [x for x in (args.layered_sizes or "small,medium,large").split(",") if x]
@@ -423,6 +461,8 @@ def run(args) -> None:
     return run_tunavik(args, sizes, prompts, hbm, tf, src)
   if getattr(args, "layered_family", "") == "fubelorn":
     return run_fubelorn(args, sizes, prompts, hbm, tf, src)
+  if getattr(args, "layered_family", "") == "fekanex":
+    return run_fekanex(args, sizes, prompts, hbm, tf, src)
   if getattr(args, "layered_family", "") == "rinutar":
     return run_rinutar(args, sizes, prompts, hbm, tf, src)
   for name in sizes:
