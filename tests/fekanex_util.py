@@ -23,7 +23,7 @@ def yarn(factor=8.0, original=40, fast=6.0, slow=0.5):
   return {"factor": float(factor), "original": original, "fast": float(fast), "slow": float(slow)}
 
 
-def attn(heads=4, kv_heads=2, dim=12, vdim=10, conv: Optional[int] = 3, rot_dims=8, base=100.0, scaling: Optional[dict] = None, size: Optional[int] = 9, keep=2,
+def attn(heads=4, kv_heads=2, dim=12, vdim=12, conv: Optional[int] = 3, rot_dims=8, base=100.0, scaling: Optional[dict] = None, size: Optional[int] = 9, keep=2,
          scale=None, v_mix=False, mlp=None):
   """one layer; rot_dims 0 = no rotation, size None = no window"""
   m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv, "scale": float(scale if scale is not None else dim ** -0.5), "v_mix": bool(v_mix),

@@ -43,6 +43,7 @@ SINGLE = {
   "many_heads": ([attn(heads=40, kv_heads=20, dim=4, vdim=4, rot_dims=4)], {}),
   "odd_sizes": ([attn(heads=3, kv_heads=3, dim=5, vdim=7, rot_dims=4)], {"width": 37}),
   "unit_sizes": ([attn(heads=1, kv_heads=1, dim=1, vdim=1, rot_dims=0)], {}),
+  "heads_beyond_128": ([attn(heads=2, kv_heads=1, dim=200, vdim=140, rot_dims=150, base=1e4, scaling=yarn()), attn(heads=1, kv_heads=1, dim=132, vdim=8, conv=4)], {}),
   "wide_heads": ([attn(heads=2, kv_heads=1, dim=272, vdim=140, rot_dims=200, base=1e4)], {}),
   "wide_values": ([attn(heads=2, kv_heads=1, vdim=300)], {}),
   "no_filter": ([attn(conv=None)], {}),
@@ -63,8 +64,15 @@ SINGLE = {
   "kept_tokens_beyond_window": ([attn(size=3, keep=8)], {}),
   "window_beyond_prompt": ([attn(size=500, keep=2)], {}),
   "no_window": ([attn(size=None)], {}),
+  # head sizes that are no multiple of 4 take the preparation kernel for any size, the others mostly the one in fours
+  "plain_filter": ([attn(vdim=10)], {}),
+  "plain_no_filter": ([attn(vdim=10, conv=None)], {}),
+  "plain_filter_2": ([attn(dim=10, conv=2)], {}),
+  "plain_yarn": ([attn(vdim=9, rot_dims=12, scaling=yarn())], {}),
+  "plain_values_mixed": ([attn(vdim=10, v_mix=True), attn(vdim=10, v_mix=True)], {}),
+  "rotated_part_no_multiple_of_4": ([attn(rot_dims=6), attn(rot_dims=10, scaling=yarn()), attn(rot_dims=2)], {}),
   "values_mixed": ([attn(v_mix=True), attn(v_mix=True)], {}),
-  "values_mixed_later": ([attn(vdim=6), attn(v_mix=True), attn(kv_heads=1), attn(heads=2, dim=8, v_mix=True)], {}),
+  "values_mixed_later": ([attn(vdim=8), attn(v_mix=True), attn(kv_heads=1), attn(heads=2, dim=8, v_mix=True)], {}),
   "dense": ([attn(mlp=dense(36))], {}),
   "dense_aligned": ([attn(mlp=dense(64))], {}),
   "dense_odd": ([attn(mlp=dense(29))], {}),
@@ -156,11 +164,12 @@ def test_first_tokens_of_a_sequence(dtype):
 
 # ---- state between steps made to stand out -----------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("vdim", [8, 9])
 @pytest.mark.parametrize("taps", [2, 4, 10])
-def test_filters_that_only_see_the_oldest_input(taps, dtype):
+def test_filters_that_only_see_the_oldest_input(taps, vdim, dtype):
   """every filter is a pure delay by taps - 1 tokens, so a token's queries, keys and values come wholly from earlier steps' inputs when it
   is decoded; portions shorter than the filter move part of the inputs on"""
-  cfg = config([attn(conv=taps, v_mix=True), attn(conv=taps, v_mix=True)])
+  cfg = config([attn(vdim=vdim, conv=taps, v_mix=True), attn(vdim=vdim, conv=taps, v_mix=True)])
   W = fo.random_weights(cfg, 6)
   for k in W:
     if k.endswith(".conv"):
@@ -605,7 +614,7 @@ def test_inference_engine_serves_a_model_directory(tmp_path):
   import asyncio
   from xotorch_b200.inference.b200_engine import B200ShardInferenceEngine, LocalDirDownloader
   from xotorch_b200.inference.shard import Shard
-  cfg = config([attn(v_mix=True, mlp=dense(36)), attn(heads=2, dim=10, v_mix=False), attn(v_mix=True, mlp=dense(20))])
+  cfg = config([attn(vdim=10, v_mix=True, mlp=dense(36)), attn(heads=2, dim=10, v_mix=False), attn(vdim=10, v_mix=True, mlp=dense(20))])
   W = fo.random_weights(cfg, 27)
   write_model_dir(tmp_path, cfg, W)
   n = len(cfg["layers"])

@@ -1182,13 +1182,33 @@ static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout)
     a.rot_dims = s.rot_dims; a.rot_layout = s.rot_layout; a.rot_mul = L.rot_mul;
     a.state = e->state + L.conv_off; a.state_slot_stride = e->state_floats;
     a.vfirst = e->vfirst; a.vmix_mode = L.vmix_mode;
-    // stretches of one row group each; as many heads per block as still leave a few blocks for every SM
+    // stretches of one row group each
     const int zs = std::max(1, std::min(65535, cdiv(sp.max_rows, GQA_PREP_ROWS)));
-    a.spc = (int)std::max<long>(1, std::min<long>(8, (long)cdiv(M, GQA_PREP_ROWS) * slots / (8L * e->sm_count)));
-    const size_t psm = (size_t)GQA_PREP_ROWS * (dk + s.rot_dims) * 4;
-    auto pk = gqa_filter_prepare_kernel<T>;
-    TRY(opt_in_smem(pk, psm));
-    pk<<<dim3(sp.n_seq, cdiv(slots, a.spc), zs), 128, psm, e->stream>>>(a, sp.seqs, pg, pool, e->qfull, q16);
+    float* qf = sp.items.at(-gqa_rows_per_item(s)).second > 0 ? e->qfull : nullptr;   // fp32 queries: read by the warp-per-(row, head) kernel alone
+    const int taps = std::max(1, s.conv_taps), hmax = std::max(dk, dv);
+    const bool vec = dk % 4 == 0 && dv % 4 == 0 && hmax <= 256 && taps <= 4 && (s.rot_dims == 0 || s.rot_layout == XOTB200_LM_ROT_INTERLEAVED) &&
+                     (L.ld_in | L.c_q | L.c_kk | L.c_vv) % 4 == 0 && (taps == 1 || (L.conv_off % 4 == 0 && e->state_floats % 4 == 0));
+    if (vec) {
+      const size_t vsm = (size_t)GQA_PREP_VEC_ROWS * ((s.rot_dims + 3) & ~3) * 4;
+      const dim3 grid(sp.n_seq, cdiv(slots, 8), zs);
+#define LAUNCH_PREP(TAPS)                                                                                                          \
+  do {                                                                                                                             \
+    if (hmax <= 128) gqa_filter_prepare_vec_kernel<T, TAPS, 1><<<grid, 256, vsm, e->stream>>>(a, sp.seqs, pg, pool, qf, q16);      \
+    else gqa_filter_prepare_vec_kernel<T, TAPS, 2><<<grid, 256, vsm, e->stream>>>(a, sp.seqs, pg, pool, qf, q16);                  \
+  } while (0)
+      if (taps == 1) LAUNCH_PREP(1);
+      else if (taps == 2) LAUNCH_PREP(2);
+      else if (taps == 3) LAUNCH_PREP(3);
+      else LAUNCH_PREP(4);
+#undef LAUNCH_PREP
+    } else {
+      // as many heads per block as still leave a few blocks for every SM
+      a.spc = (int)std::max<long>(1, std::min<long>(8, (long)cdiv(M, GQA_PREP_ROWS) * slots / (8L * e->sm_count)));
+      const size_t psm = (size_t)GQA_PREP_ROWS * (dk + s.rot_dims) * 4;
+      auto pk = gqa_filter_prepare_kernel<T>;
+      TRY(opt_in_smem(pk, psm));
+      pk<<<dim3(sp.n_seq, cdiv(slots, a.spc), zs), 128, psm, e->stream>>>(a, sp.seqs, pg, pool, qf, q16);
+    }
   } else {
     gqa_prepare_kernel<T><<<cdiv((long)M * slots, 8), 256, 0, e->stream>>>(
         e->proj, L.ld_in, L.c_q, L.c_kk, L.c_vv, s.proj_bias ? at<T>(e, L.b_in) : nullptr, weighted ? at<T>(e, L.q_norm) : nullptr,

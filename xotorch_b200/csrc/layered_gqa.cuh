@@ -22,7 +22,8 @@
 // Queries may carry a temperature: the query at position p is multiplied by 1 + coef * ln(1 + (p + 1) / every), integer quotient.
 //
 // Kernels: gqa_prepare_kernel (bias, per-head RMS norm, temperature, cache append), gqa_prepare_row_kernel (the same with ONE norm
-// over the whole query / key projection), gqa_filter_prepare_kernel (the same with short convolutions, norm after rotation, mixed values), gqa_attention_kernel + gqa_combine_kernel (one warp per (row, query head); decode,
+// over the whole query / key projection), gqa_filter_prepare_kernel / gqa_filter_prepare_vec_kernel (the same with
+// short convolutions, norm after rotation, mixed values), gqa_attention_kernel + gqa_combine_kernel (one warp per (row, query head); decode,
 // short portions and the 32-bit mode), gqa_flash_kernel (tensor cores, bf16, long portions).
 #pragma once
 #include "layered_kernels.cuh"
@@ -196,7 +197,7 @@ __global__ void gqa_prepare_row_kernel(const float* __restrict__ proj, int ld, i
 // The same step for layers with any of: short causal convolutions on the projections, a head norm AFTER the rotation, a rotation whose
 // cosines and sines carry a factor, values mixed with an earlier layer's.  In order, per row and channel:
 //   u = proj + bias;  f = sum_{j < taps} w[c, j] u(pos - taps + 1 + j)    (no filter when taps == 0; u of earlier steps from `state`)
-//   q, k: head norm (norm_when 1) -> rotation (times rot_mul) -> head norm (norm_when 2) -> query temperature -> qf / q16, pool
+//   q, k: head norm (norm_when 1) -> rotation (times rot_mul) -> head norm (norm_when 2) -> query temperature -> qf, q16 (either may be NULL) / pool
 //   v   : vmix_mode 1: f is also kept in vfirst [M, G * dv];  2: (1 - c) f + c vfirst, c = *vmix;  -> pool
 // grid (requests, groups of `spc` head slots, row stretches).  A stretch is at least taps - 1 rows, so only stretch 0 reads a slot's
 // filter inputs ([taps - 1][C] fp32 at `state`, zero at the start of a request) — and the threads that read a channel move its inputs on
@@ -206,6 +207,7 @@ __global__ void gqa_prepare_row_kernel(const float* __restrict__ proj, int ld, i
 // Dynamic shared memory: GQA_PREP_ROWS * (dk + rot_dims) floats.
 // ---------------------------------------------------------------------------------------------------------------------------
 constexpr int GQA_PREP_ROWS = 8, GQA_PREP_TAPS = 8;   // rows per group; taps up to which weights and the sliding window stay in registers
+constexpr int GQA_PREP_VEC_ROWS = 4;                  // rows a lane of the kernel in fours holds at once (3 blocks per SM: 80 registers)
 
 struct GqaPrep {
   const float* proj;
@@ -343,7 +345,7 @@ __global__ void __launch_bounds__(128) gqa_filter_prepare_kernel(const GqaPrep a
           const size_t o = ((size_t)(sq.row0 + t0 + r) * H + hd) * dk;
           for (int d = lane; d < dk; d += 32) {
             const float v = f[d] * fac * (a.norm_when == 2 && w ? ldf(w + d) : 1.f);
-            qf[o + d] = v;
+            if (qf) qf[o + d] = v;
             if (q16) q16[o + d] = __float2bfloat16_rn(v);
           }
         } else {
@@ -354,6 +356,202 @@ __global__ void __launch_bounds__(128) gqa_filter_prepare_kernel(const GqaPrep a
       __syncthreads();                                         // the next head overwrites fs
     }
   }
+}
+
+// four neighbouring entries of T, on a boundary of four
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld4(const bf16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162 *a = reinterpret_cast<const __nv_bfloat162*>(&r.x), *b = reinterpret_cast<const __nv_bfloat162*>(&r.y);
+  const float2 x = __bfloat1622float2(*a), y = __bfloat1622float2(*b);
+  return make_float4(x.x, x.y, y.x, y.y);
+}
+__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w)); }
+
+// The same for the sizes most models have: head sizes that are multiples of 4 (<= 128 * NV), TAPS taps (1 = also "no filter"), pairs
+// (2i, 2i + 1) rotated or no rotation, everything on boundaries of four.  One warp owns one head for a stretch of rows: a lane holds four
+// neighbouring channels (both members of two planes), their filter weights and the sliding window in registers, so a head needs no
+// shared memory and no block barrier; only the rotation's cosines and sines are shared, by the eight heads of the block.
+// grid (requests, groups of 8 head slots, row stretches), 256 threads; dynamic shared memory: GQA_PREP_VEC_ROWS * (rot_dims up to a
+// multiple of 4) floats.
+template <typename T, int TAPS, int NV>
+__global__ void __launch_bounds__(256, NV == 1 ? 3 : 2) gqa_filter_prepare_vec_kernel(const GqaPrep a, const Item* __restrict__ seqs, Paging pg, T* __restrict__ pool, float* __restrict__ qf,
+                                                                     bf16* __restrict__ q16) {
+  extern __shared__ __align__(16) float cs[];                  // [RB][rs]: cosine, sine of every plane
+  constexpr int KEEP = TAPS - 1, RB = GQA_PREP_VEC_ROWS / NV;  // rows held at once
+  __shared__ size_t prow[RB];                                  // their places in the pool
+  const Item sq = seqs[blockIdx.x];
+  const int H = a.H, G = a.G, dk = a.dk, dv = a.dv, C = H * dk + (a.own_kv ? G * (dk + dv) : 0), slots = H + (a.own_kv ? 2 * G : 0);
+  const int per = max((sq.n_rows + (int)gridDim.z - 1) / (int)gridDim.z, max(KEEP, 1));
+  const int t_begin = blockIdx.z * per, t_end = min(sq.n_rows, t_begin + per);
+  if (t_begin >= t_end) return;
+  const int sl = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const bool active = sl < slots, is_q = sl < H, is_v = sl >= H + G;
+  const int hd = is_q ? sl : is_v ? sl - H - G : sl - H, dim = is_v ? dv : dk;
+  const int c0 = (is_q ? a.col_q : is_v ? a.col_v : a.col_k) + hd * dim, half = a.rot_dims >> 1, rs = (a.rot_dims + 3) & ~3;
+  const size_t rowlen = (size_t)G * (dk + dv);
+  const T *bias = static_cast<const T*>(a.bias), *cw = static_cast<const T*>(a.conv_w), *w = static_cast<const T*>(is_q ? a.q_norm : a.k_norm);
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), one = make_float4(1.f, 1.f, 1.f, 1.f);
+  float* st = KEEP > 0 ? a.state + (size_t)sq.slot * a.state_slot_stride : nullptr;
+  const float* pr = a.proj + (size_t)sq.row0 * a.ld + c0;
+  float4 bs[NV], nw[NV], wt[NV][TAPS], win[NV][KEEP > 0 ? KEEP : 1];
+  int dd[NV];
+  bool on[NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int d = (v * 32 + lane) * 4;
+    dd[v] = d;
+    on[v] = active && d < dim;
+    bs[v] = on[v] && bias ? ld4(bias + c0 + d) : zero;
+    nw[v] = on[v] && w && !is_v ? ld4(w + d) : one;
+    const int ch = c0 + d - a.col_q;
+    if (on[v] && cw) {
+      float t[4 * TAPS];
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) { const float4 q = ld4(cw + (size_t)ch * TAPS + 4 * i); t[4 * i] = q.x; t[4 * i + 1] = q.y; t[4 * i + 2] = q.z; t[4 * i + 3] = q.w; }
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) wt[v][i] = make_float4(t[i], t[TAPS + i], t[2 * TAPS + i], t[3 * TAPS + i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) wt[v][i] = one;           // TAPS == 1 without a filter: times one
+    }
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int r = t_begin - KEEP + i;
+      win[v][i] = !on[v] ? zero : r >= 0 ? add4(ld4(pr + (size_t)r * a.ld + d), bs[v]) : ld4(st + (size_t)(r + KEEP) * C + ch);
+    }
+  }
+  const float vm = a.vmix_mode == 2 ? ldf(static_cast<const T*>(a.vmix)) : 0.f;
+  for (int t0 = t_begin; t0 < t_end; t0 += RB) {
+    const int n = min(RB, t_end - t0);
+    float4 f[RB][NV];                                          // the projection's rows, then what becomes of them; rows past n are never stored
+#pragma unroll
+    for (int i = 0; i < RB; ++i)
+#pragma unroll
+      for (int v = 0; v < NV; ++v) f[i][v] = on[v] && i < n ? ld4(pr + (size_t)(t0 + i) * a.ld + dd[v]) : zero;
+    if (t0 > t_begin) __syncthreads();                         // the last rows' tables are no longer read
+    if (threadIdx.x >= 224 && threadIdx.x - 224 < n) prow[threadIdx.x - 224] = pg.row(sq.slot, sq.pos0 + t0 + (int)threadIdx.x - 224) * rowlen;
+    if (a.freqs)
+      for (int i = threadIdx.x; i < n * half; i += blockDim.x) {
+        const int r = i / half, p = i - r * half;
+        float sn, cn;
+        sincosf((float)(sq.pos0 + t0 + r) * a.freqs[p], &sn, &cn);
+        *reinterpret_cast<float2*>(cs + r * rs + 2 * p) = make_float2(cn * a.rot_mul, sn * a.rot_mul);
+      }
+    __syncthreads();
+    if (!active) continue;
+#pragma unroll
+    for (int i = 0; i < RB; ++i)
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const float4 u = on[v] ? add4(f[i][v], bs[v]) : zero;
+        float4 y = zero;
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) y = fma4(wt[v][j], win[v][j], y);
+        f[i][v] = fma4(wt[v][KEEP], u, y);
+#pragma unroll
+        for (int j = 0; j + 1 < KEEP; ++j) win[v][j] = win[v][j + 1];
+        if (KEEP > 0) win[v][KEEP > 0 ? KEEP - 1 : 0] = u;
+      }
+    if (is_v) {
+      float* vf = a.vmix_mode ? a.vfirst + ((size_t)sq.row0 + t0) * (G * dv) + (size_t)hd * dv : nullptr;
+      if (a.vmix_mode == 2) {
+#pragma unroll
+        for (int i = 0; i < RB; ++i)
+#pragma unroll
+          for (int v = 0; v < NV; ++v)
+            if (on[v] && i < n) f[i][v] = add4(scale4(f[i][v], 1.0f - vm), scale4(ld4(vf + (size_t)i * (G * dv) + dd[v]), vm));
+      }
+#pragma unroll
+      for (int i = 0; i < RB; ++i)
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+          if (!on[v] || i >= n) continue;
+          if (a.vmix_mode == 1) st4(vf + (size_t)i * (G * dv) + dd[v], f[i][v]);
+          st4(pool + prow[i] + (size_t)G * dk + (size_t)hd * dv + dd[v], f[i][v]);
+        }
+      continue;
+    }
+    // 1 / root mean square of every row's head; the rows' reductions go side by side
+    auto head_scales = [&](float (&s)[RB]) {
+#pragma unroll
+      for (int i = 0; i < RB; ++i) {
+        s[i] = 0.f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) s[i] = fmaf(f[i][v].x, f[i][v].x, fmaf(f[i][v].y, f[i][v].y, fmaf(f[i][v].z, f[i][v].z, fmaf(f[i][v].w, f[i][v].w, s[i]))));
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < RB; ++i) s[i] += __shfl_xor_sync(0xffffffffu, s[i], o);
+#pragma unroll
+      for (int i = 0; i < RB; ++i) s[i] = 1.0f / sqrtf(s[i] / (float)dk + a.eps);
+    };
+    float s[RB];
+    if (a.norm_when == 1) {
+      head_scales(s);
+#pragma unroll
+      for (int i = 0; i < RB; ++i)
+#pragma unroll
+        for (int v = 0; v < NV; ++v) f[i][v] = mul4(scale4(f[i][v], s[i]), nw[v]);
+    }
+    if (a.freqs) {
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        if (dd[v] >= a.rot_dims) continue;
+        const bool both = dd[v] + 2 < a.rot_dims;              // rot_dims may end between the lane's two planes
+#pragma unroll
+        for (int i = 0; i < RB; ++i) {
+          const float4 c = *reinterpret_cast<const float4*>(cs + (i < n ? i : 0) * rs + dd[v]), g = f[i][v];
+          f[i][v].x = g.x * c.x - g.y * c.y;
+          f[i][v].y = g.y * c.x + g.x * c.y;
+          if (both) {
+            f[i][v].z = g.z * c.z - g.w * c.w;
+            f[i][v].w = g.w * c.z + g.z * c.w;
+          }
+        }
+      }
+    }
+    if (a.norm_when == 2) {
+      head_scales(s);
+#pragma unroll
+      for (int i = 0; i < RB; ++i)
+#pragma unroll
+        for (int v = 0; v < NV; ++v) f[i][v] = mul4(scale4(f[i][v], s[i]), nw[v]);
+    }
+#pragma unroll
+    for (int i = 0; i < RB; ++i) {
+      if (i >= n) break;
+      const float fac = is_q ? gqa_query_temperature(a.q_temp_coef, a.q_temp_every, sq.pos0 + t0 + i) : 1.0f;
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        if (!on[v]) continue;
+        const float4 y = scale4(f[i][v], fac);
+        if (is_q) {
+          const size_t o = (((size_t)sq.row0 + t0 + i) * H + hd) * dk + dd[v];
+          if (qf) st4(qf + o, y);
+          if (q16) st4(q16 + o, y);
+        } else {
+          st4(pool + prow[i] + (size_t)hd * dk + dd[v], y);
+        }
+      }
+    }
+  }
+  if (KEEP > 0 && blockIdx.z == 0)
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      if (!on[v]) continue;
+      const int ch = c0 + dd[v] - a.col_q;
+      for (int i = 0; i < KEEP; ++i) {                         // increasing i: entry i + n_rows is still the old one when it is read
+        const int r = sq.n_rows - KEEP + i;
+        st4(st + (size_t)i * C + ch, r >= 0 ? add4(ld4(pr + (size_t)r * a.ld + dd[v]), bs[v]) : ld4(st + (size_t)(i + sq.n_rows) * C + ch));
+      }
+    }
 }
 
 // table[a][d] = rel[bucket_of[d], a] for d < n: the learned bias of head a at distance d (rel is [buckets, H] as stored)
