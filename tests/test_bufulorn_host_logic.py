@@ -43,7 +43,7 @@ def test_c_structs_mirror_the_header():
   for name, cls in (("xotb200_lm_layer", _lib.LmLayer), ("xotb200_lm_cfg", _lib.LmCfg)):
     body = re.search(r"typedef struct " + name + r" \{(.*?)\} " + name + ";", src, re.S).group(1)
     body = re.sub(r"/\*.*?\*/", "", body, flags=re.S)
-    fields = re.findall(r"\b(?:int32_t|float)\s+(\w+)\s*;", body)
+    fields = re.findall(r"\b(?:int32_t|int64_t|float)\s+(\w+)\s*;", body)
     assert fields == [f for f, _ in cls._fields_]
 
 

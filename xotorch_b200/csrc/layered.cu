@@ -1254,7 +1254,8 @@ static int gqa_layer(xotb200_lm* e, LmLayer& L, const StepPlan& sp, float* yout)
     CK(cudaGetLastError());
     e->launches++;
     if (splits > 1) {
-      gqa_combine_kernel<T><<<dim3(it.second, cdiv(qpi * H, 8)), 256, 0, e->stream>>>(e->part, it.first, H, dv, splits, static_cast<const T*>(sc.sink), sc.sink_one, gate, s.out_gate, L.ld_in, L.c_g, static_cast<T*>(e->oh));
+      // few pairs: their value columns are cut over grid.z
+      gqa_combine_kernel<T><<<dim3(it.second, cdiv(qpi * H, 8), it.second * cdiv(qpi * H, 8) < 4 * e->sm_count ? cdiv(dv, 32) : 1), 256, 0, e->stream>>>(e->part, it.first, H, dv, splits, static_cast<const T*>(sc.sink), sc.sink_one, gate, s.out_gate, L.ld_in, L.c_g, static_cast<T*>(e->oh));
       CK(cudaGetLastError());
       e->launches++;
     }

@@ -698,7 +698,7 @@ __global__ void gqa_attention_kernel(const float* __restrict__ qf, const T* __re
   }
 }
 
-// merges the key runs: one warp per (row, query head) of the listed items; at most 32 runs.  A sink (per head, or of score 0 for all with
+// merges the key runs: one warp per (row, query head) of the listed items (grid.y covers the pairs) and 32-column piece (grid.z); at most 32 runs.  A sink (per head, or of score 0 for all with
 // sink_one) joins here, once, like a run that holds the weight exp(sink) and no values.
 template <typename T>
 __global__ void gqa_combine_kernel(const float* __restrict__ part, const Item* __restrict__ items, int H, int dv, int splits, const T* __restrict__ sink,
@@ -715,7 +715,7 @@ __global__ void gqa_combine_kernel(const float* __restrict__ part, const Item* _
   const float wz = mz == -INFINITY ? 0.f : expf(mz - mx);
   const float den = warp_sum(lane < splits ? src[(size_t)lane * (2 + dv) + 1] * wz : 0.f) + (sink || sink_one ? expf(sk - mx) : 0.f);
   const float inv = 1.0f / den;
-  for (int d0 = 0; d0 < dv; d0 += 32) {
+  for (int d0 = blockIdx.z * 32; d0 < dv; d0 += 32 * gridDim.z) {
     const int d = d0 + lane;
     float a = 0.f;
 #pragma unroll 8
