@@ -225,7 +225,7 @@ def fekanex_config(s: dict, b: dict):
   moe = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP}, "expert": {"ff": s["ff"] // 4}}
   layers = [{"type": "attention", "mixer": mixer, "mlp": mlp} for _ in range(3 * s["repeats"] // 2) for mlp in (dense, moe)]
   cfg = {"architecture": "Fekanex", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
-         "embedding": {"scale": 2.0, "bigram": {"buckets": FEK_BUCKETS, "mul_prev": 10007, "mul_cur": 31}}, "layers": layers}
+         "embedding": {"scale": 2.0, "bigram": {"buckets": FEK_BUCKETS, "mul_prev": 10007, "mul_cur": 13}}, "layers": layers}
   return cfg, len(layers) // 2 * (EXPERTS - TOP) * 3 * (s["ff"] // 4) * s["width"] * 2
 
 
